@@ -3,6 +3,7 @@ from .fusitar import FusitarConfig
 from .gemma2 import ConfigError, Gemma2Config
 from .kofutar import KofutarConfig
 from .lokedra import LokedraConfig
+from .mukunex import MukunexConfig
 from .teluzen import TeluzenConfig
 from .registry import (
     architectures,
@@ -17,6 +18,7 @@ from .registry import (
 from .spec import (
     AttentionSpec,
     BlockSpec,
+    ChannelDeltaSpec,
     DeltaSpec,
     EmbedSpec,
     ForgetGateSpec,
@@ -25,6 +27,7 @@ from .spec import (
     HeadSpec,
     InputAddSpec,
     InputMixSpec,
+    LRUSpec,
     LatentAttentionSpec,
     MLPSpec,
     MLSTMSpec,
@@ -33,6 +36,8 @@ from .spec import (
     NormSpec,
     ParallelMixerSpec,
     PositionSpec,
+    RetentionSpec,
+    RopeBands,
     RopeScaling,
     ScheduleEntry,
     default_schedule,

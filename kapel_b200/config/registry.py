@@ -16,6 +16,7 @@ from .fusitar import FusitarConfig
 from .gemma2 import ConfigError, Gemma2Config
 from .kofutar import KofutarConfig
 from .lokedra import LokedraConfig
+from .mukunex import MukunexConfig
 from .teluzen import TeluzenConfig
 
 _ARCHITECTURES: Dict[str, type] = {}
@@ -104,3 +105,4 @@ register_architecture(FusitarConfig, FusitarConfig.architecture, FusitarConfig.m
 register_architecture(KofutarConfig, KofutarConfig.architecture, KofutarConfig.model_type)
 register_architecture(TeluzenConfig, TeluzenConfig.architecture, TeluzenConfig.model_type)
 register_architecture(LokedraConfig, LokedraConfig.architecture, LokedraConfig.model_type)
+register_architecture(MukunexConfig, MukunexConfig.architecture, MukunexConfig.model_type)

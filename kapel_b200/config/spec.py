@@ -41,17 +41,30 @@ class RopeScaling:
 
 
 @dataclass(frozen=True)
+class RopeBands:
+    """Frequencies slowed by wavelength in three bands (as Llama 3.1 does): with wavelength l = 2 pi / f a
+    frequency is kept where l < original / high, divided by `factor` where l > original / low, and between
+    the two it is (1 - s) f / factor + s f with s = (original / l - low) / (high - low)."""
+
+    factor: float
+    low: float
+    high: float
+    original: float
+
+
+@dataclass(frozen=True)
 class PositionSpec:
     """kind "rope": rotation of the first `rotary_dim` components, pairing "half" (j, j+r/2) or
     "neighbours" (2j, 2j+1), by the angle position * theta^(-2j/r) / `divisor` (a divisor above 1
-    stretches the positions); with `scaling` the frequencies follow `RopeScaling` instead."""
+    stretches the positions); with `scaling` the frequencies follow that record's rule (`RopeScaling` or
+    `RopeBands`) instead."""
 
     kind: str = "rope"
     theta: float = 10000.0
     rotary_dim: int = 0
     pairing: str = "half"
     divisor: float = 1.0
-    scaling: Optional[RopeScaling] = None
+    scaling: Optional[object] = None
 
 
 @dataclass(frozen=True)
@@ -86,6 +99,9 @@ class AttentionSpec:
     floor(j / B), blocks counted from position 0. `unit_sink`: 1 joins the softmax's denominator (a key
     of score 0 without a value). `out_bias`: o has a bias (role o_bias); with `qk_bias` q and k have
     biases and v has none.
+
+    `sink`: e^(sink[head]) joins the softmax's denominator (role sink [heads]; no key, no value, not scaled).
+    `gate_by_head` (with `gated`): the gate is one number a head (g [heads, hidden]).
     """
 
     hidden: int
@@ -118,6 +134,8 @@ class AttentionSpec:
     unit_sink: bool = False
     qk_bias: bool = False
     out_bias: bool = False
+    sink: bool = False
+    gate_by_head: bool = False
 
 
 @dataclass(frozen=True)
@@ -172,6 +190,72 @@ class DeltaSpec:
     weights: Mapping[str, str]
     unit_eps: float = 1e-6
     kind: str = "delta"
+
+
+@dataclass(frozen=True)
+class ChannelDeltaSpec:
+    """The gated delta rule with a decay a head and key channel (`DeltaSpec`'s is one a head).
+
+    q, k, v, their convolutions, silu, unit vectors and beta = sigmoid(b h) as `DeltaSpec`; the decay
+    g = exp(-exp(A_log[head]) softplus(a2 (a1 h) + dt_bias)), laid out [heads, head_dim], through a rank of
+    `decay_rank`. Per row: S <- diag(g) S; u = beta (v - S^T k); S <- S + k u^T; o = S^T q. Each head's o
+    is divided by its root mean square (`eps`), times the weight `norm` [v_head_dim] (one for all heads),
+    times sigmoid(g2 (g1 h)) laid out [heads, v_head_dim] (a rank of `gate_rank`), then o. `weights`: q, k,
+    v, q_conv, k_conv, v_conv, b, A_log, a1, a2, dt_bias, norm, g1, g2, o.
+    """
+
+    hidden: int
+    num_heads: int
+    num_kv_heads: int
+    head_dim: int
+    v_head_dim: int
+    conv: int
+    decay_rank: int
+    gate_rank: int
+    eps: float
+    weights: Mapping[str, str]
+    unit_eps: float = 1e-6
+    kind: str = "channel_delta"
+
+
+@dataclass(frozen=True)
+class RetentionSpec:
+    """Linear attention with a fixed decay a head (retention): a matrix memory S [head_dim, v_head_dim] a
+    head and request.
+
+    q, k [heads, head_dim] turned by `position`, k then times head_dim^-1/2; v [heads, v_head_dim].
+    S <- `decay`[head] S + k v^T; o = S^T q, no softmax and no denominator. Each head's o is divided by its
+    root mean square (`eps`, no weight), times silu(g h), then o. `weights`: q, k, v, g, o.
+    """
+
+    hidden: int
+    num_heads: int
+    head_dim: int
+    v_head_dim: int
+    decay: Tuple[float, ...]
+    eps: float
+    position: PositionSpec
+    weights: Mapping[str, str]
+    kind: str = "retention"
+
+
+@dataclass(frozen=True)
+class LRUSpec:
+    """A real-gated linear recurrent unit between two branches of `width` channels (Griffin's recurrent block).
+
+    y = gelu_tanh(y h + y_bias); u = conv(x h + x_bias) + conv_bias, a causal convolution over `conv` rows
+    per channel. u in `blocks` equal parts: r = sigmoid(ra[b] u_b + ra_bias[b]), i = sigmoid(ri[b] u_b +
+    ri_bias[b]). a = exp(-`rate` r softplus(lam)); S <- a S + sqrt(1 - a^2) i u channel by channel; the
+    output is o (S y). `weights`: y, y_bias, x, x_bias, conv, conv_bias, ra, ra_bias, ri, ri_bias, lam, o.
+    """
+
+    hidden: int
+    width: int
+    blocks: int
+    conv: int
+    weights: Mapping[str, str]
+    rate: float = 8.0
+    kind: str = "rglru"
 
 
 @dataclass(frozen=True)

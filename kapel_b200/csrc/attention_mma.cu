@@ -59,7 +59,7 @@ struct AttMmaParams {
     int window, split, slots;
     int keep;                  // with a window: keys [0, keep) stay visible below it (prompt kernel only, one slot)
     int block;                 // > 0: a row at position i sees only the keys from floor(i / block) * block on (prompt kernel only, one slot)
-    const float* sinks;        // [hq] or null: e^sink joins a row's denominator (prompt kernel only, one slot)
+    const float* sinks;        // [hq] or null: e^sink joins a row's denominator (once: where a row's slots are merged)
     int decode_bar_offset;     // bytes from the start of shared memory to the decode kernel's mbarriers
     int direct;                // 1: a row whose keys all lie in one slot was written to `out` by that slot's block
     int relative;              // 1: every request brings one token (tile t = row t = request t) and slots are counted from the row's first visible key, else from key 0
@@ -948,6 +948,12 @@ attention_decode_kernel(const AttMmaParams p, const __grid_constant__ CUtensorMa
         }
         const int row = row0 + r / group, head = kvh * group + r % group;
         if (p.slots == 1) {
+            if (p.sinks != nullptr) {
+                const float sink = p.sinks[head], top = fmaxf(mx, sink);
+                const float wk = mx == -INFINITY ? 0.f : __expf(mx - top);
+                acc *= wk;
+                l = fmaf(l, wk, __expf(sink - top));
+            }
             p.out[((size_t)row * p.hq + head) * d + c] = __float2bfloat16_rn(l > 0.f ? acc / l : 0.f);
         } else {
             float* dst = p.partial + (((size_t)row * p.hq + head) * p.slots + slot) * (d + 2);
@@ -1005,6 +1011,7 @@ attention_mma_combine_kernel(const AttMmaParams p KB_TL_PARAM) {
         }
         for (int z = lane + 128; z < nz; z += 32) mx = fmaxf(mx, base[(size_t)z * stride + p.d]);
         mx = warp_max(mx);
+        if (p.sinks != nullptr) mx = fmaxf(mx, p.sinks[head]);
         float denom = 0.f;
 #pragma unroll
         for (int j = 0; j < 4; ++j) {
@@ -1022,6 +1029,7 @@ attention_mma_combine_kernel(const AttMmaParams p KB_TL_PARAM) {
             denom += w * base[(size_t)z * stride + p.d + 1];
         }
         denom = warp_sum(denom);
+        if (p.sinks != nullptr) denom += __expf(p.sinks[head] - mx);
         const float inv = denom > 0.f ? 1.f / denom : 0.f;
         for (int z = lane; z < nz; z += 32) cw[z] *= inv;
     }
@@ -1111,6 +1119,7 @@ attention_mma_combine_bulk_kernel(const AttMmaParams p KB_TL_PARAM) {
         float mx = -INFINITY;
         for (int z = lane; z < nz; z += 32) mx = fmaxf(mx, base[(size_t)z * stride + p.d]);
         mx = warp_max(mx);
+        if (p.sinks != nullptr) mx = fmaxf(mx, p.sinks[head]);
         float denom = 0.f;
         for (int z = lane; z < nz; z += 32) {
             const float m = base[(size_t)z * stride + p.d];
@@ -1119,6 +1128,7 @@ attention_mma_combine_bulk_kernel(const AttMmaParams p KB_TL_PARAM) {
             denom += w * base[(size_t)z * stride + p.d + 1];
         }
         denom = warp_sum(denom);
+        if (p.sinks != nullptr) denom += __expf(p.sinks[head] - mx);
         const float inv = denom > 0.f ? 1.f / denom : 0.f;
         for (int z = lane; z < nz; z += 32) cw[z] *= inv;
     }
@@ -1169,6 +1179,7 @@ attention_mma_combine_warp_kernel(const AttMmaParams p) {
     float mx = -INFINITY;
     for (int z = lane; z < nz; z += 32) mx = fmaxf(mx, base[(size_t)z * stride + p.d]);
     mx = warp_max(mx);
+    if (p.sinks != nullptr) mx = fmaxf(mx, p.sinks[head]);
     float denom = 0.f;
     for (int z = lane; z < nz; z += 32) {
         const float m = base[(size_t)z * stride + p.d];
@@ -1177,6 +1188,7 @@ attention_mma_combine_warp_kernel(const AttMmaParams p) {
         denom += w * base[(size_t)z * stride + p.d + 1];
     }
     denom = warp_sum(denom);
+    if (p.sinks != nullptr) denom += __expf(p.sinks[head] - mx);
     const float inv = denom > 0.f ? 1.f / denom : 0.f;
     __syncwarp();
     for (int i = lane * 2; i < p.d; i += 64) {              // d and the stride are even
@@ -1370,8 +1382,8 @@ extern "C" int kb_attention_mma_masked(void* out, const void* q, const void* k_t
     KB_REQUIRE(hkv <= 65535, "attention_mma: %d kv heads is too many for one launch", hkv);
     KB_REQUIRE(keep >= 0 && (keep == 0 || (window > 0 && !decode && split == 0 && slots == 1)),
                "attention_mma: %d first keys kept need a window, prompt portions and one slot", keep);
-    KB_REQUIRE(block >= 0 && ((block == 0 && sinks == nullptr) || (!decode && split == 0 && slots == 1 && keep == 0)),
-               "attention_mma: a block mask (%d) or sinks need prompt portions, one slot and no kept first keys", block);
+    KB_REQUIRE(block >= 0 && (block == 0 || (!decode && split == 0 && slots == 1 && keep == 0)),
+               "attention_mma: a block mask (%d) needs prompt portions, one slot and no kept first keys", block);
     if (rows == 0 || tiles == 0) return 0;
     AttMmaParams p;
     p.keep = keep; p.block = block; p.sinks = sinks;

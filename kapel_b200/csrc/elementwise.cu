@@ -535,6 +535,34 @@ extern "C" int kb_pad_cols_bf16(void* out, const void* in, long long rows, int w
     return check_launch("pad_cols");
 }
 
+// out[r, 0:n] = x[r, off : off + n] of a product (a tensor or split-K partial sums), zeros behind it up to `wide`.
+template <typename TI, typename TO>
+__global__ void take_cols_kernel(TO* __restrict__ out, const Src<TI> x, int row_width, int off, int n, int wide, long long total) {
+    const long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
+    if (i >= total) return;
+    const long long r = i / wide;
+    const int c = (int)(i - r * wide);
+    Elem<TO>::store(out + i, c < n ? x.at((size_t)r * row_width + off + c) : 0.f);
+}
+
+extern "C" int kb_take_cols(void* out, int out_dt, const void* x, int in_dt, int splits, long long split_stride, int row_width, int off,
+                            int n, int wide, long long rows, void* stream) {
+    KB_REQUIRE(rows >= 0 && n > 0 && wide >= n && off >= 0 && off + (long long)n <= row_width, "take_cols: columns %d (+%d, to %d) of a row of %d", off, n, wide, row_width);
+    KB_REQUIRE(splits >= 1 && (splits == 1 || split_stride >= rows * row_width), "take_cols: %d slices %lld apart", splits, split_stride);
+    if (rows == 0) return 0;
+    const long long total = rows * wide;
+    KB_REQUIRE((total + 255) / 256 <= 0x7fffffffll, "take_cols: too many values for one launch");
+    const unsigned blocks = (unsigned)((total + 255) / 256);
+    cudaStream_t s = (cudaStream_t)stream;
+#define KB_TC(TI, TO) take_cols_kernel<TI, TO><<<blocks, 256, 0, s>>>((TO*)out, Src<TI>{(const TI*)x, splits, (size_t)split_stride}, row_width, off, n, wide, total)
+    if (in_dt == KB_DT_F32 && out_dt == KB_DT_F32) KB_TC(float, float);
+    else if (in_dt == KB_DT_F32 && out_dt == KB_DT_BF16) KB_TC(float, bf16);
+    else if (in_dt == KB_DT_BF16 && out_dt == KB_DT_BF16) KB_TC(bf16, bf16);
+    else return fail("take_cols: dtype codes %d -> %d are not known", in_dt, out_dt);
+#undef KB_TC
+    return check_launch("take_cols");
+}
+
 // out[r, :] = (a[r, :], b[r, :]) side by side, float32 in, `out_dt` out.
 template <typename TO>
 __global__ void concat2_kernel(TO* __restrict__ out, const float* __restrict__ a, const float* __restrict__ b, long long rows, int width) {

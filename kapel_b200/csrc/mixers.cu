@@ -6,8 +6,9 @@
 //                    [rows, hq, d], keys and values written to the paged cache at each row's line.
 //                    The counterpart of rotate-and-append for a mixer without a rotation.
 //  head_gate         y[r, h, :] (optionally divided by its root mean square over the head, times a
-//                    weight over all heads) times sigmoid(gate[r, h, :]), the gate read from the
-//                    stacked product; the output's rows may be wider than the heads (zeros behind them).
+//                    weight over all heads) times sigmoid(gate[r, h, :]) (or one gate a head), the gate read
+//                    from the stacked product, times a number; the output's rows may be wider than the heads
+//                    (zeros behind them) and the heads may start at a later column.
 //  entry_ranges      first row and one past the last row of every request of a step, from the rows' entries.
 //  head_norm_rope_append  an RMS norm over every head's query and key (a weight of the head's size,
 //                    shared by the heads), then the rotation of the first `rotary` components, the
@@ -81,7 +82,7 @@ __global__ void proj_norm_append_kernel(const Src<TS> src, int row_width, int q_
 template <typename TY, typename TS, typename TW, typename TO>
 __global__ void head_gate_kernel(TO* __restrict__ out, const TY* __restrict__ y, const Src<TS> gate, int row_width,
                                  int g_off, const TW* __restrict__ w, int unit, float eps, long long pairs, int heads, int e,
-                                 int out_stride, int act) {
+                                 int out_stride, int fill_to, int act, int by_head, float scale) {
     const long long pair = (long long)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
     if (pair >= pairs) return;
     const int lane = threadIdx.x & 31;
@@ -98,10 +99,15 @@ __global__ void head_gate_kernel(TO* __restrict__ out, const TY* __restrict__ y,
         ss = warp_sum(ss);
         inv = 1.f / sqrtf(ss / (float)e + eps);
     }
+    inv *= scale;
+    if (by_head && act != 2) {                                                   // one gate for the whole head
+        const float z = gate.at((size_t)r * row_width + g_off + h);
+        inv *= act == 1 ? z / (1.f + expf(-z)) : 1.f / (1.f + expf(-z));
+    }
     for (int c = lane; c < e; c += 32) {
         float v = Elem<TY>::load(yp + c) * inv;
         if (w != nullptr) v *= Elem<TW>::load(w + (size_t)h * e + c);
-        if (act != 2) {                                                          // 2: no gate
+        if (act != 2 && !by_head) {                                              // 2: no gate
             const float z = gate.at((size_t)r * row_width + g_off + (size_t)h * e + c);
             v *= act == 1 ? z / (1.f + expf(-z)) : 1.f / (1.f + expf(-z));       // silu(z) or sigmoid(z)
         }
@@ -109,7 +115,7 @@ __global__ void head_gate_kernel(TO* __restrict__ out, const TY* __restrict__ y,
     }
     // a row wider than its heads (padding for the product that follows) ends in zeros
     if (h == heads - 1)
-        for (int c = heads * e + lane; c < out_stride; c += 32) Elem<TO>::store(out + (size_t)r * out_stride + c, 0.f);
+        for (int c = heads * e + lane; c < fill_to; c += 32) Elem<TO>::store(out + (size_t)r * out_stride + c, 0.f);
 }
 
 // One block a row; a warp takes head vectors in turn (queries, then keys, then values) through a
@@ -513,11 +519,13 @@ extern "C" int kb_proj_norm_append(const void* src, int in_dt, int splits, long 
 
 extern "C" int kb_head_gate(void* out, int out_dt, const void* y, int y_dt, const void* gate, int g_dt, int splits,
                             long long split_stride, int row_width, int g_off, const void* w, int w_dt, int unit, float eps,
-                            long long rows, int heads, int e, int out_stride, int act, void* stream) {
+                            long long rows, int heads, int e, int out_stride, int fill_to, int act, int by_head, float scale, void* stream) {
+    // out: the first of this call's columns in rows `out_stride` apart; zeros go behind the heads up to column `fill_to`
     KB_REQUIRE(rows >= 0 && heads > 0 && e > 0, "head_gate: rows %lld, heads %d of %d", rows, heads, e);
+    KB_REQUIRE(fill_to >= heads * e && fill_to <= out_stride, "head_gate: %d heads of %d filled to column %d in rows of %d", heads, e, fill_to, out_stride);
     KB_REQUIRE(act >= 0 && act <= 2, "head_gate: gate activation code %d is not known (0 sigmoid, 1 silu, 2 none)", act);
     KB_REQUIRE(out_stride >= heads * e, "head_gate: output rows of %d values for %d heads of %d", out_stride, heads, e);
-    KB_REQUIRE(row_width > 0 && g_off >= 0 && g_off + heads * e <= row_width, "head_gate: gate columns %d.. do not fit a row of %d", g_off, row_width);
+    KB_REQUIRE(row_width > 0 && g_off >= 0 && g_off + heads * (by_head ? 1 : e) <= row_width, "head_gate: gate columns %d.. do not fit a row of %d", g_off, row_width);
     KB_REQUIRE(splits >= 1 && (splits == 1 || split_stride >= rows * row_width), "head_gate: %d slices %lld apart", splits, split_stride);
     if (rows == 0) return 0;
     cudaStream_t s = (cudaStream_t)stream;
@@ -528,7 +536,7 @@ extern "C" int kb_head_gate(void* out, int out_dt, const void* y, int y_dt, cons
 #define KB_HG(TY, TS, TW, TO)                                                                                       \
     head_gate_kernel<TY, TS, TW, TO><<<(unsigned)blocks, warps * 32, 0, s>>>((TO*)out, (const TY*)y,                    \
                                                                              Src<TS>{(const TS*)gate, splits, (size_t)split_stride}, \
-                                                                             row_width, g_off, (const TW*)w, unit, eps, pairs, heads, e, out_stride, act)
+                                                                             row_width, g_off, (const TW*)w, unit, eps, pairs, heads, e, out_stride, fill_to, act, by_head, scale)
     const int code = y_dt * 8 + g_dt * 4 + w_dt * 2 + out_dt;
     switch (code) {
         case 0: KB_HG(float, float, float, float); break;

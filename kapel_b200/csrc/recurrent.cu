@@ -13,9 +13,12 @@
 //                        S <- diag(w) S - b (u^T S) + k v^T,   o = S^T r      (both first terms read the old S)
 //                    Written on the old memory: with p = u^T S and q = (w r)^T S, o = q - p (b.r) + v (k.r),
 //                    so both dot products of a row are reduced together. `gdelta_prep` (the generalized
-//                    delta rule: decay through a small two-layer net, removal rate, unit keys) and
+//                    delta rule: decay through a small two-layer net, removal rate, unit keys),
 //                    `gate_prep` (tied gates: a forget gate with a lower bound, and one minus it as the input gate:
-//                    w = f, k = 1 - f, no removal) make its inputs.
+//                    w = f, k = 1 - f, no removal), `cdelta_prep` (the gated delta rule with a decay a key channel:
+//                    S <- diag(w) S + b (v - p)^T, o = q + (v - p) (b.r)) and `retention_prep` (a fixed decay a
+//                    head, rotated queries and keys) make its inputs.
+//  conv_rows         the convolution alone: a bias, the filter, another bias, written out in 32-bit.
 //  weighted_sum2     out = a * va + b * vb + vc with a weight a channel on each branch.
 //
 // Everything here is 32-bit; only the projections may come in bfloat16.
@@ -70,6 +73,7 @@ struct ConvParams {
     int row_width, q_off, k_off, nq, nk;      // columns of the stacked product; nq = hq d, nk = hkv d
     const float* bias;                        // [nq + nk] or null
     const float* conv;                        // [nq + nk, taps]: the last weight is the row's own
+    const float* after;                       // [nq + nk] or null: added behind the filter
     float* state;                             // [slots, (taps - 1) (nq + nk)]
     const int* row_entry;
     const int* entry_start;
@@ -111,6 +115,7 @@ __global__ void conv_append_kernel(const Src<TS> src, const ConvParams p, TO* __
             else x = 0.f;
             y = fmaf(p.conv[(size_t)c * p.taps + (p.taps - 1 - j)], x, y);
         }
+        if (p.after != nullptr) y += p.after[c];
         if (is_q) {
             Elem<TO>::store(q_out + (size_t)r * p.q_stride + c, y);
         } else {
@@ -151,8 +156,8 @@ __global__ void conv_history_kernel(const Src<TS> src, const ConvParams p) {
 }
 
 // ------------------------------------------------------------------------------------------ the scan's inputs
-// Scratch of a step: vectors [rows, heads, NV, d] in the order (w r, w, k, u, b) (NV = 5 with the removal,
-// else the first 3), values [rows, heads, e], scalars [rows, heads, 2] = (b.r, k.r).
+// Scratch of a step: vectors [rows, heads, NV, d] as the scan's mode lists them below, values [rows, heads, e],
+// scalars [rows, heads, 2] = (b.r, k.r).
 struct ScanInputs {
     float* vec;
     float* val;
@@ -280,7 +285,183 @@ gate_prep_kernel(const Src<TS> src, const GateParams p, const ScanInputs s) {
     for (int i = threadIdx.x; i < nv; i += blockDim.x) s.val[(size_t)r * nv + i] = src.at(base + p.v_off + i);
 }
 
+struct CDeltaParams {
+    int row_width, q_off, k_off, v_off, b_off, a1_off, rank;
+    const float* a2;            // [rank, heads d]: the decay's second factor turned, so that neighbouring threads read neighbouring weights
+    const float* dt_bias;       // [heads d]
+    const float* a_log;         // [heads]
+    const float* conv;          // [2 kv_heads d + heads e, taps]: q's channels, then k's, then v's
+    const float* state;         // [slots, (taps - 1) channels]: the convolutions' last inputs
+    const int* row_entry;
+    const int* entry_start;
+    const int* slots;
+    int n_slots, entries, heads, kv_heads, d, e, taps;
+    float q_scale, unit_eps;
+};
+
+__device__ __forceinline__ float rc_softplus(float x) { return x > 20.f ? x : log1pf(expf(x)); }
+
+// The convolution and silu of one channel of a row: the inputs before the step come from the request's history.
+template <typename TS>
+__device__ __forceinline__ float conv_silu(const Src<TS>& src, const CDeltaParams& p, int r, int r0, const float* hist, int channels, int col, int c) {
+    float y = 0.f;
+    for (int j = 0; j < p.taps; ++j) {                          // the input j rows back
+        const int t = r - j;
+        float x = 0.f;
+        if (t >= r0) x = src.at((size_t)t * p.row_width + col);
+        else if (hist != nullptr) x = hist[(size_t)(p.taps - 1 + (t - r0)) * channels + c];
+        y = fmaf(p.conv[(size_t)c * p.taps + (p.taps - 1 - j)], x, y);
+    }
+    return y * rc_sigmoid(y);
+}
+
+// One block RB rows. The decay of every (head, key channel) is a thread's: exp(-exp(A_log) softplus(a2 . hidden + dt_bias)), its
+// column of a2 read once for the block's rows; a warp a (row, head) then convolves that head's query and key, makes them unit
+// vectors and leaves (g q, g, beta k, g k) and beta k.q; a thread a channel the values.
+template <typename TS, int RB>
+__global__ void __launch_bounds__(1024)
+cdelta_prep_kernel(const Src<TS> src, const CDeltaParams p, const ScanInputs s, int rows) {
+    extern __shared__ float hid[];                              // [RB][rank]
+    const int r0 = blockIdx.x * RB;
+    const int nr = min(RB, rows - r0);
+    const int d = p.d, n = p.heads * d, nq = p.kv_heads * d, nv = p.heads * p.e;
+    const int channels = 2 * nq + nv;
+    for (int idx = threadIdx.x; idx < RB * p.rank; idx += blockDim.x) {
+        const int rr = idx / p.rank, j = idx - rr * p.rank;
+        hid[idx] = rr < nr ? src.at((size_t)(r0 + rr) * p.row_width + p.a1_off + j) : 0.f;
+    }
+    __syncthreads();
+    for (int c = threadIdx.x; c < n; c += blockDim.x) {
+        float z[RB];
+#pragma unroll
+        for (int rr = 0; rr < RB; ++rr) z[rr] = 0.f;
+        for (int j = 0; j < p.rank; ++j) {
+            const float wj = p.a2[(size_t)j * n + c];
+#pragma unroll
+            for (int rr = 0; rr < RB; ++rr) z[rr] = fmaf(wj, hid[rr * p.rank + j], z[rr]);
+        }
+        const float bias = p.dt_bias[c];
+        const int h = c / d, i = c - h * d;
+        const float rate = expf(p.a_log[h]);
+#pragma unroll
+        for (int rr = 0; rr < RB; ++rr)
+            if (rr < nr) s.vec[((size_t)(r0 + rr) * p.heads + h) * 4 * d + d + i] = expf(-rate * rc_softplus(z[rr] + bias));
+    }
+    __syncthreads();
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, warps = blockDim.x >> 5;
+    const int per = p.heads / p.kv_heads;
+    for (int pair = warp; pair < nr * p.heads; pair += warps) {
+        const int rr = pair / p.heads, h = pair - rr * p.heads;
+        const int r = r0 + rr, kvh = h / per;
+        const int entry = p.row_entry[r];
+        const bool known = entry >= 0 && entry < p.entries;
+        const int first = known ? p.entry_start[entry] : r;
+        const int slot = known ? p.slots[entry] : 0;
+        const float* hist = slot > 0 && slot < p.n_slots ? p.state + (size_t)slot * (p.taps - 1) * channels : nullptr;
+        float q[8], k[8];                                       // d <= 256
+        float sq = 0.f, sk = 0.f;
+#pragma unroll
+        for (int x = 0; x < 8; ++x) {
+            const int i = lane + 32 * x;
+            q[x] = k[x] = 0.f;
+            if (i < d) {
+                const int c = kvh * d + i;
+                q[x] = conv_silu(src, p, r, first, hist, channels, p.q_off + c, c);
+                k[x] = conv_silu(src, p, r, first, hist, channels, p.k_off + c, nq + c);
+                sq = fmaf(q[x], q[x], sq);
+                sk = fmaf(k[x], k[x], sk);
+            }
+        }
+        sq = warp_sum(sq);
+        sk = warp_sum(sk);
+        const float iq = p.q_scale / sqrtf(sq + p.unit_eps), ik = 1.f / sqrtf(sk + p.unit_eps);
+        const float beta = rc_sigmoid(src.at((size_t)r * p.row_width + p.b_off + h));
+        float* vec = s.vec + ((size_t)r * p.heads + h) * 4 * d;
+        float br = 0.f;
+#pragma unroll
+        for (int x = 0; x < 8; ++x) {
+            const int i = lane + 32 * x;
+            if (i < d) {
+                const float g = vec[d + i], qn = q[x] * iq, kn = k[x] * ik;
+                vec[i] = g * qn;
+                vec[2 * d + i] = beta * kn;
+                vec[3 * d + i] = g * kn;
+                br = fmaf(beta * kn, qn, br);
+            }
+        }
+        br = warp_sum(br);
+        if (lane == 0) {
+            s.scal[((size_t)r * p.heads + h) * 2] = br;
+            s.scal[((size_t)r * p.heads + h) * 2 + 1] = 0.f;
+        }
+    }
+    for (int idx = threadIdx.x; idx < nr * nv; idx += blockDim.x) {
+        const int rr = idx / nv, c = idx - rr * nv;
+        const int r = r0 + rr;
+        const int entry = p.row_entry[r];
+        const bool known = entry >= 0 && entry < p.entries;
+        const int first = known ? p.entry_start[entry] : r;
+        const int slot = known ? p.slots[entry] : 0;
+        const float* hist = slot > 0 && slot < p.n_slots ? p.state + (size_t)slot * (p.taps - 1) * channels : nullptr;
+        s.val[(size_t)r * nv + c] = conv_silu(src, p, r, first, hist, channels, p.v_off + c, 2 * nq + c);
+    }
+}
+
+struct RetentionParams {
+    int row_width, q_off, k_off, v_off;
+    const float* decay;         // [heads]
+    const float2* cos_sin;      // [rows, rotary / 2]
+    int rotary, heads, d, e;
+    float k_scale;
+};
+
+// One block a row, a warp a head: queries and keys turned (component i with i + rotary / 2), keys scaled; the scan's inputs
+// are decay q and k.
+template <typename TS>
+__global__ void __launch_bounds__(256)
+retention_prep_kernel(const Src<TS> src, const RetentionParams p, const ScanInputs s) {
+    const int r = blockIdx.x;
+    const size_t base = (size_t)r * p.row_width;
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, warps = blockDim.x >> 5;
+    const int half = p.rotary >> 1, d = p.d;
+    for (int h = warp; h < p.heads; h += warps) {
+        float kr = 0.f;
+        const float decay = p.decay[h];
+        float* vec = s.vec + ((size_t)r * p.heads + h) * 2 * d;
+        auto put = [&](int i, float q, float k) {
+            k *= p.k_scale;
+            vec[i] = decay * q;
+            vec[d + i] = k;
+            kr = fmaf(k, q, kr);
+        };
+        const size_t qa = base + p.q_off + (size_t)h * d, ka = base + p.k_off + (size_t)h * d;
+        for (int i = lane; i < half; i += 32) {
+            float q0 = src.at(qa + i), q1 = src.at(qa + half + i), k0 = src.at(ka + i), k1 = src.at(ka + half + i);
+            const float2 cs = p.cos_sin[(size_t)r * half + i];
+            rope_rotate(q0, q1, cs);
+            rope_rotate(k0, k1, cs);
+            put(i, q0, k0);
+            put(half + i, q1, k1);
+        }
+        for (int i = 2 * half + lane; i < d; i += 32) put(i, src.at(qa + i), src.at(ka + i));
+        kr = warp_sum(kr);
+        if (lane == 0) {
+            s.scal[((size_t)r * p.heads + h) * 2] = 0.f;
+            s.scal[((size_t)r * p.heads + h) * 2 + 1] = kr;
+        }
+    }
+    const int nv = p.heads * p.e;
+    for (int i = threadIdx.x; i < nv; i += blockDim.x) s.val[(size_t)r * nv + i] = src.at(base + p.v_off + i);
+}
+
 // ------------------------------------------------------------------------------------------ the scan
+// What the vectors of a row are, and what a row does:
+//   SCAN_GATE     (w r, w, k)         S <- diag(w) S + k v^T
+//   SCAN_REMOVAL  (w r, w, k, u, b)   S <- diag(w) S - b (u^T S) + k v^T
+//   SCAN_WRITE    (w r, w, b, u)      S <- diag(w) S + b (v - u^T S)^T
+//   SCAN_FIXED    (w r, k)            S <- w S + k v^T with one w a head
+enum ScanMode { SCAN_GATE = 0, SCAN_REMOVAL = 1, SCAN_WRITE = 2, SCAN_FIXED = 3 };
+__host__ __device__ constexpr int scan_vectors(int mode) { return mode == SCAN_REMOVAL ? 5 : (mode == SCAN_WRITE ? 4 : (mode == SCAN_FIXED ? 2 : 3)); }
 constexpr int SC = 4;                  // warps a block
 constexpr int SCAN_R = 8;              // memory rows a lane can hold: d <= 32 * SCAN_R
 
@@ -288,6 +469,7 @@ struct ScanParams {
     const float* vec;           // [rows, heads, NV, d]
     const float* val;           // [rows, heads, e]
     const float* scal;          // [rows, heads, 2]
+    const float* fixed;         // [heads] the decay of SCAN_FIXED
     float* state;               // [slots, heads, e, d]: a column of a head's memory lies together
     const int* entry_start;
     const int* entry_end;
@@ -325,11 +507,12 @@ __device__ __forceinline__ void scan_load(float (&dst)[R], const float* p) {
 
 // One block = one request of the step x one head x SC * DW columns of the memory; a warp DW columns, lane l
 // the rows R l .. R l + R - 1 of them in registers (a row's vectors then come from shared memory 16 bytes a load). R: rows a lane holds; CH: rows of the step staged at a time
-// (asynchronous copies, the next chunk while this one is walked); REMOVAL: whether u and b exist.
-template <int R, int CH, int DW, bool REMOVAL>
+// (asynchronous copies, the next chunk while this one is walked).
+template <int R, int CH, int DW, int MODE>
 __global__ void __launch_bounds__(SC * 32)
 decay_scan_kernel(const ScanParams p) {
-    constexpr int NV = REMOVAL ? 5 : 3;
+    constexpr int NV = scan_vectors(MODE);
+    constexpr bool TWO_SUMS = MODE == SCAN_REMOVAL || MODE == SCAN_WRITE;      // p = u^T S beside q
     constexpr int DP = R * 32;
     constexpr int COLS = SC * DW;
     constexpr int tail = NV * DP;                               // v [COLS] | b.r | k.r | padding
@@ -394,6 +577,7 @@ decay_scan_kernel(const ScanParams p) {
         }
     }
     const bool hi16 = lane & 16;
+    const float fixed = MODE == SCAN_FIXED ? p.fixed[head] : 0.f;
     const int chunks = (r1 - r0 + CH - 1) / CH;
     stage(0, 0);
     for (int ch = 0; ch < chunks; ++ch) {
@@ -410,19 +594,21 @@ decay_scan_kernel(const ScanParams p) {
         for (int t = 0; t < nr; ++t) {
             const float* in = rows + (size_t)t * rowf;
             const float br = in[tail + COLS], kr = in[tail + COLS + 1];
-            float wr[R], w[R], k[R], u[REMOVAL ? R : 1], b[REMOVAL ? R : 1];
+            float wr[R], w[R], k[R], u[TWO_SUMS ? R : 1], b[MODE == SCAN_REMOVAL ? R : 1];
             scan_load<R>(wr, in + lane * R);
-            scan_load<R>(w, in + DP + lane * R);
-            scan_load<R>(k, in + 2 * DP + lane * R);
-            if constexpr (REMOVAL) {
-                scan_load<R>(u, in + 3 * DP + lane * R);
-                scan_load<R>(b, in + 4 * DP + lane * R);
+            if constexpr (MODE == SCAN_FIXED) {
+                scan_load<R>(k, in + DP + lane * R);
+            } else {
+                scan_load<R>(w, in + DP + lane * R);
+                scan_load<R>(k, in + 2 * DP + lane * R);
             }
+            if constexpr (TWO_SUMS) scan_load<R>(u, in + 3 * DP + lane * R);
+            if constexpr (MODE == SCAN_REMOVAL) scan_load<R>(b, in + 4 * DP + lane * R);
 #pragma unroll
             for (int ci = 0; ci < DW; ++ci) {
                 const float v = in[tail + warp * DW + ci];
                 float o;
-                if constexpr (REMOVAL) {
+                if constexpr (TWO_SUMS) {
                     float xp = 0.f, xq = 0.f;
 #pragma unroll
                     for (int i = 0; i < R; ++i) {
@@ -438,15 +624,22 @@ decay_scan_kernel(const ScanParams p) {
                     y += __shfl_xor_sync(0xffffffffu, y, 2);
                     y += __shfl_xor_sync(0xffffffffu, y, 1);
                     const float pp = __shfl_sync(0xffffffffu, y, 0), qq = __shfl_sync(0xffffffffu, y, 16);
+                    if constexpr (MODE == SCAN_REMOVAL) {
 #pragma unroll
-                    for (int i = 0; i < R; ++i) S[ci][i] = fmaf(k[i], v, fmaf(-b[i], pp, w[i] * S[ci][i]));
-                    o = fmaf(v, kr, fmaf(-pp, br, qq));
+                        for (int i = 0; i < R; ++i) S[ci][i] = fmaf(k[i], v, fmaf(-b[i], pp, w[i] * S[ci][i]));
+                        o = fmaf(v, kr, fmaf(-pp, br, qq));
+                    } else {
+                        const float x = v - pp;
+#pragma unroll
+                        for (int i = 0; i < R; ++i) S[ci][i] = fmaf(k[i], x, w[i] * S[ci][i]);
+                        o = fmaf(x, br, qq);
+                    }
                 } else {
                     float xq = 0.f;
 #pragma unroll
                     for (int i = 0; i < R; ++i) {
                         xq = fmaf(S[ci][i], wr[i], xq);
-                        S[ci][i] = fmaf(k[i], v, w[i] * S[ci][i]);
+                        S[ci][i] = fmaf(k[i], v, (MODE == SCAN_FIXED ? fixed : w[i]) * S[ci][i]);
                     }
                     xq = warp_sum(xq);
                     o = fmaf(v, kr, xq);
@@ -521,7 +714,7 @@ extern "C" int kb_conv_append(void* q_out, int q_stride, void* k_table, int out_
     KB_REQUIRE(entries <= 65535, "conv_append: too many requests for one launch");
     if (rows == 0 || entries == 0) return 0;
     ConvParams p;
-    p.row_width = row_width; p.q_off = q_off; p.k_off = k_off; p.nq = nq; p.nk = nk; p.bias = bias; p.conv = conv; p.state = state;
+    p.row_width = row_width; p.q_off = q_off; p.k_off = k_off; p.nq = nq; p.nk = nk; p.bias = bias; p.conv = conv; p.after = nullptr; p.state = state;
     p.row_entry = row_entry; p.entry_start = entry_start; p.entry_end = entry_end; p.slots = slots; p.lines = lines;
     p.n_slots = n_slots; p.entries = entries; p.rows = rows; p.taps = taps; p.hkv = hkv; p.d = d; p.page_size = page_size;
     p.q_stride = q_stride; p.table_lines = table_lines;
@@ -545,9 +738,9 @@ extern "C" int kb_conv_append(void* q_out, int q_stride, void* k_table, int out_
     return check_launch("conv_append history");
 }
 
-// Floats of scratch for a step of `rows` rows of the scan: the vectors, the values, the two scalars.
-extern "C" long long kb_decay_scan_scratch_floats(int rows, int heads, int d, int e, int removal) {
-    return (long long)rows * heads * ((removal ? 5ll : 3ll) * d + e + 2);
+// Floats of scratch for a step of `rows` rows of the scan in this mode: the vectors, the values, the two scalars.
+extern "C" long long kb_decay_scan_scratch_floats(int rows, int heads, int d, int e, int mode) {
+    return (long long)rows * heads * ((long long)scan_vectors(mode) * d + e + 2);
 }
 
 // 0: the launcher chooses how many columns of the memory a warp of the scan holds; 1 or 2: that many (for tests and measurements).
@@ -555,8 +748,9 @@ static int g_scan_columns = 0;
 extern "C" void kb_decay_scan_columns(int n) { g_scan_columns = (n == 1 || n == 2 || n == 4) ? n : 0; }
 
 static int run_decay_scan(float* out, const ScanInputs& in, float* state, int n_slots, const int* entry_start, const int* entry_end,
-                          const int* slots, int entries, int heads, int d, int e, bool removal, cudaStream_t s) {
+                          const int* slots, int entries, int heads, int d, int e, int mode, const float* fixed, cudaStream_t s) {
     ScanParams p;
+    p.fixed = fixed;
     p.vec = in.vec; p.val = in.val; p.scal = in.scal; p.state = state; p.entry_start = entry_start; p.entry_end = entry_end;
     p.slots = slots; p.n_slots = n_slots; p.heads = heads; p.d = d; p.e = e; p.out = out;
     int sms = 148;
@@ -571,23 +765,26 @@ static int run_decay_scan(float* out, const ScanInputs& in, float* state, int n_
     KB_REQUIRE((e + SC * dw - 1) / (SC * dw) <= 65535 && heads <= 65535, "decay_scan: too many heads or value components for one launch");
     dim3 grid(entries, heads, (e + SC * dw - 1) / (SC * dw));
     const int need = (d + 31) / 32;
-#define KB_SCAN(R, CH, W, REM)                                                                                    \
+#define KB_SCAN(R, CH, W, MODE)                                                                                   \
     do {                                                                                                          \
-        const size_t smem = (size_t)2 * CH * ((REM ? 5 : 3) * R * 32 + SC * W + 4) * sizeof(float);               \
-        if (smem > 48 * 1024) cudaFuncSetAttribute(decay_scan_kernel<R, CH, W, REM>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
-        decay_scan_kernel<R, CH, W, REM><<<grid, SC * 32, smem, s>>>(p);                                          \
+        const size_t smem = (size_t)2 * CH * (scan_vectors(MODE) * R * 32 + SC * W + 4) * sizeof(float);          \
+        if (smem > 48 * 1024) cudaFuncSetAttribute(decay_scan_kernel<R, CH, W, MODE>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
+        decay_scan_kernel<R, CH, W, MODE><<<grid, SC * 32, smem, s>>>(p);                                         \
     } while (0)
-#define KB_SCAN_W(R, CH)                                  \
-    do {                                                  \
-        if (removal) {                                    \
-            if (dw == 4) KB_SCAN(R, CH, (R <= 4 ? 4 : 2), true);      \
-            else if (dw == 2) KB_SCAN(R, CH, 2, true);    \
-            else KB_SCAN(R, CH, 1, true);                 \
-        } else {                                          \
-            if (dw == 4) KB_SCAN(R, CH, (R <= 4 ? 4 : 2), false);     \
-            else if (dw == 2) KB_SCAN(R, CH, 2, false);   \
-            else KB_SCAN(R, CH, 1, false);                \
-        }                                                 \
+#define KB_SCAN_M(R, CH, MODE)                                        \
+    do {                                                              \
+        if (dw == 4) KB_SCAN(R, CH, (R <= 4 ? 4 : 2), MODE);          \
+        else if (dw == 2) KB_SCAN(R, CH, 2, MODE);                    \
+        else KB_SCAN(R, CH, 1, MODE);                                 \
+    } while (0)
+#define KB_SCAN_W(R, CH)                                              \
+    do {                                                              \
+        switch (mode) {                                               \
+            case SCAN_REMOVAL: KB_SCAN_M(R, CH, SCAN_REMOVAL); break; \
+            case SCAN_WRITE: KB_SCAN_M(R, CH, SCAN_WRITE); break;     \
+            case SCAN_FIXED: KB_SCAN_M(R, CH, SCAN_FIXED); break;     \
+            default: KB_SCAN_M(R, CH, SCAN_GATE); break;              \
+        }                                                             \
     } while (0)
     if (need <= 1) KB_SCAN_W(1, 16);
     else if (need <= 2) KB_SCAN_W(2, 16);
@@ -600,6 +797,7 @@ static int run_decay_scan(float* out, const ScanInputs& in, float* state, int n_
         KB_SCAN_W(SCAN_R, 4);
     }
 #undef KB_SCAN_W
+#undef KB_SCAN_M
 #undef KB_SCAN
     return check_launch("decay_scan");
 }
@@ -655,7 +853,7 @@ extern "C" int kb_gdelta_scan(float* out, float* scratch, const void* src, int i
     else return fail("gdelta: dtype code %d is not known", in_dt);
 #undef KB_GD
     if (int err = check_launch("gdelta prep")) return err;
-    return run_decay_scan(out, in, state, n_slots, entry_start, entry_end, slots, entries, heads, d, d, true, s);
+    return run_decay_scan(out, in, state, n_slots, entry_start, entry_end, slots, entries, heads, d, d, SCAN_REMOVAL, nullptr, s);
 }
 
 // The read-out [rows, heads, e] of the memory behind a forget gate with a lower bound.
@@ -683,7 +881,125 @@ extern "C" int kb_gate_scan(float* out, float* scratch, const void* src, int in_
     else if (in_dt == KB_DT_BF16) gate_prep_kernel<bf16><<<rows, 256, 0, s>>>(Src<bf16>{(const bf16*)src, splits, (size_t)split_stride}, g, in);
     else return fail("gate_scan: dtype code %d is not known", in_dt);
     if (int err = check_launch("gate_scan prep")) return err;
-    return run_decay_scan(out, in, state, n_slots, entry_start, entry_end, slots, entries, heads, d, e, false, s);
+    return run_decay_scan(out, in, state, n_slots, entry_start, entry_end, slots, entries, heads, d, e, SCAN_GATE, nullptr, s);
+}
+
+// The read-out [rows, heads, e] of the gated delta rule with a decay a key channel; `history` [slots, (taps - 1) channels]
+// holds the convolutions' last inputs and `memory` [slots, heads, e, d] the memories.
+extern "C" int kb_cdelta_scan(float* out, float* scratch, const void* src, int in_dt, int splits, long long split_stride, int row_width,
+                              int q_off, int k_off, int v_off, int b_off, int a1_off, int rank, const float* a2, const float* dt_bias,
+                              const float* a_log, const float* conv, float* history, float* memory, int n_slots, const int* row_entry,
+                              const int* entry_start, const int* entry_end, const int* slots, int entries, int rows, int heads,
+                              int kv_heads, int d, int e, int taps, float q_scale, float unit_eps, void* stream) {
+    if (int err = scan_common_checks("cdelta", src, splits, split_stride, row_width, rows, entries, heads, d, e, memory, n_slots, entry_start, entry_end, slots))
+        return err;
+    KB_REQUIRE(kv_heads > 0 && heads % kv_heads == 0, "cdelta: %d heads over %d", heads, kv_heads);
+    KB_REQUIRE(taps >= 1 && taps <= CONV_MAX_TAPS, "cdelta: a convolution of %d taps (1 to %d)", taps, CONV_MAX_TAPS);
+    const long long nq = (long long)kv_heads * d, nv = (long long)heads * e, n = (long long)heads * d;
+    KB_REQUIRE(row_width > 0 && q_off >= 0 && k_off == q_off + nq && v_off == k_off + nq && v_off + nv <= row_width,
+               "cdelta: columns q %d, k %d, v %d must follow one another in a row of %d", q_off, k_off, v_off, row_width);
+    KB_REQUIRE(b_off >= 0 && b_off + heads <= row_width && rank > 0 && a1_off >= 0 && a1_off + rank <= row_width,
+               "cdelta: columns b %d, a1 %d (+%d) do not fit a row of %d", b_off, a1_off, rank, row_width);
+    KB_REQUIRE(out && scratch && a2 && dt_bias && a_log && conv && history && row_entry, "cdelta: weights, history or scratch are missing");
+    const bool few = rows <= DEPENDENT_ROWS;
+    const size_t smem = (size_t)(few ? 1 : 8) * rank * sizeof(float);
+    KB_REQUIRE(smem <= 200 * 1024, "cdelta: a decay of rank %d does not fit the shared memory of a block", rank);
+    if (entries == 0 || rows == 0) return 0;
+    CDeltaParams g;
+    g.row_width = row_width; g.q_off = q_off; g.k_off = k_off; g.v_off = v_off; g.b_off = b_off; g.a1_off = a1_off; g.rank = rank;
+    g.a2 = a2; g.dt_bias = dt_bias; g.a_log = a_log; g.conv = conv; g.state = history; g.row_entry = row_entry; g.entry_start = entry_start;
+    g.slots = slots; g.n_slots = n_slots; g.entries = entries; g.heads = heads; g.kv_heads = kv_heads; g.d = d; g.e = e; g.taps = taps;
+    g.q_scale = q_scale; g.unit_eps = unit_eps;
+    ScanInputs in;
+    in.vec = scratch;
+    in.val = in.vec + (size_t)rows * n * 4;
+    in.scal = in.val + (size_t)rows * nv;
+    in.nv = 4;
+    ConvParams c = {};
+    c.row_width = row_width; c.q_off = q_off; c.nq = (int)(2 * nq + nv); c.conv = conv; c.state = history; c.row_entry = row_entry;
+    c.entry_start = entry_start; c.entry_end = entry_end; c.slots = slots; c.n_slots = n_slots; c.entries = entries; c.rows = rows; c.taps = taps;
+    cudaStream_t s = (cudaStream_t)stream;
+#define KB_CD(TS)                                                                                                          \
+    do {                                                                                                                   \
+        const Src<TS> x{(const TS*)src, splits, (size_t)split_stride};                                                      \
+        if (few) {                                                                                                         \
+            if (smem > 48 * 1024) cudaFuncSetAttribute(cdelta_prep_kernel<TS, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
+            cdelta_prep_kernel<TS, 1><<<rows, 1024, smem, s>>>(x, g, in, rows);                                            \
+        } else {                                                                                                           \
+            if (smem > 48 * 1024) cudaFuncSetAttribute(cdelta_prep_kernel<TS, 8>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
+            cdelta_prep_kernel<TS, 8><<<(rows + 7) / 8, 512, smem, s>>>(x, g, in, rows);                                   \
+        }                                                                                                                  \
+        if (int err = check_launch("cdelta prep")) return err;                                                             \
+        if (taps > 1) conv_history_kernel<TS><<<dim3((unsigned)((c.nq + 127) / 128), entries), 128, 0, s>>>(x, c);          \
+    } while (0)
+    if (in_dt == KB_DT_F32) KB_CD(float);
+    else if (in_dt == KB_DT_BF16) KB_CD(bf16);
+    else return fail("cdelta: dtype code %d is not known", in_dt);
+#undef KB_CD
+    if (int err = check_launch("cdelta history")) return err;
+    return run_decay_scan(out, in, memory, n_slots, entry_start, entry_end, slots, entries, heads, d, e, SCAN_WRITE, nullptr, s);
+}
+
+// The read-out [rows, heads, e] of a matrix memory with a fixed decay a head behind rotated queries and keys.
+extern "C" int kb_retention_scan(float* out, float* scratch, const void* src, int in_dt, int splits, long long split_stride, int row_width,
+                                 int q_off, int k_off, int v_off, const float* decay, const float* cos_sin, int rotary, float k_scale,
+                                 float* state, int n_slots, const int* entry_start, const int* entry_end, const int* slots, int entries,
+                                 int rows, int heads, int d, int e, void* stream) {
+    if (int err = scan_common_checks("retention", src, splits, split_stride, row_width, rows, entries, heads, d, e, state, n_slots, entry_start, entry_end, slots))
+        return err;
+    const long long nq = (long long)heads * d, nv = (long long)heads * e;
+    KB_REQUIRE(row_width > 0 && q_off >= 0 && q_off + nq <= row_width && k_off >= 0 && k_off + nq <= row_width && v_off >= 0 && v_off + nv <= row_width,
+               "retention: columns q %d, k %d, v %d do not fit a row of %d", q_off, k_off, v_off, row_width);
+    KB_REQUIRE(rotary >= 0 && rotary <= d && rotary % 2 == 0 && (rotary == 0 || cos_sin), "retention: a rotation of %d components of %d", rotary, d);
+    KB_REQUIRE(out && scratch && decay, "retention: decays or scratch are missing");
+    if (entries == 0 || rows == 0) return 0;
+    RetentionParams g;
+    g.row_width = row_width; g.q_off = q_off; g.k_off = k_off; g.v_off = v_off; g.decay = decay; g.cos_sin = (const float2*)cos_sin;
+    g.rotary = rotary; g.heads = heads; g.d = d; g.e = e; g.k_scale = k_scale;
+    ScanInputs in;
+    in.vec = scratch;
+    in.val = in.vec + (size_t)rows * nq * 2;
+    in.scal = in.val + (size_t)rows * nv;
+    in.nv = 2;
+    cudaStream_t s = (cudaStream_t)stream;
+    if (in_dt == KB_DT_F32) retention_prep_kernel<float><<<rows, 256, 0, s>>>(Src<float>{(const float*)src, splits, (size_t)split_stride}, g, in);
+    else if (in_dt == KB_DT_BF16) retention_prep_kernel<bf16><<<rows, 256, 0, s>>>(Src<bf16>{(const bf16*)src, splits, (size_t)split_stride}, g, in);
+    else return fail("retention: dtype code %d is not known", in_dt);
+    if (int err = check_launch("retention prep")) return err;
+    return run_decay_scan(out, in, state, n_slots, entry_start, entry_end, slots, entries, heads, d, e, SCAN_FIXED, decay, s);
+}
+
+// out [rows, channels] = the convolution of columns off.. (bias added first, `after` behind the filter), in 32-bit; `state`
+// [slots, (taps - 1) channels] holds every request's last inputs.
+extern "C" int kb_conv_rows(float* out, const void* src, int in_dt, int splits, long long split_stride, int row_width, int off,
+                            int channels, const float* bias, const float* conv, const float* after, float* state, int n_slots,
+                            const int* row_entry, const int* entry_start, const int* entry_end, const int* slots, int entries, int rows,
+                            int taps, void* stream) {
+    KB_REQUIRE(rows >= 0 && entries >= 0 && channels > 0, "conv_rows: rows %d, requests %d, channels %d", rows, entries, channels);
+    KB_REQUIRE(taps >= 1 && taps <= CONV_MAX_TAPS, "conv_rows: a convolution of %d taps (1 to %d)", taps, CONV_MAX_TAPS);
+    KB_REQUIRE(row_width > 0 && off >= 0 && off + (long long)channels <= row_width, "conv_rows: columns %d.. do not fit a row of %d", off, row_width);
+    KB_REQUIRE(splits >= 1 && (splits == 1 || split_stride >= (long long)rows * row_width), "conv_rows: %d slices %lld apart", splits, split_stride);
+    KB_REQUIRE(out && src && conv && state && n_slots >= 1 && row_entry && entry_start && entry_end && slots, "conv_rows: a tensor is missing");
+    KB_REQUIRE(entries <= 65535, "conv_rows: too many requests for one launch");
+    if (rows == 0 || entries == 0) return 0;
+    ConvParams p = {};
+    p.row_width = row_width; p.q_off = off; p.nq = channels; p.bias = bias; p.conv = conv; p.after = after; p.state = state;
+    p.row_entry = row_entry; p.entry_start = entry_start; p.entry_end = entry_end; p.slots = slots; p.n_slots = n_slots; p.entries = entries;
+    p.rows = rows; p.taps = taps; p.q_stride = channels;
+    cudaStream_t s = (cudaStream_t)stream;
+    const int threads = channels >= 2048 ? 512 : 256;
+#define KB_CR(TS)                                                                                                          \
+    do {                                                                                                                   \
+        const Src<TS> x{(const TS*)src, splits, (size_t)split_stride};                                                      \
+        conv_append_kernel<TS, float><<<rows, threads, 0, s>>>(x, p, out, (float*)nullptr);                                 \
+        if (int err = check_launch("conv_rows")) return err;                                                               \
+        if (taps > 1) conv_history_kernel<TS><<<dim3((unsigned)((channels + 127) / 128), entries), 128, 0, s>>>(x, p);      \
+    } while (0)
+    if (in_dt == KB_DT_F32) KB_CR(float);
+    else if (in_dt == KB_DT_BF16) KB_CR(bf16);
+    else return fail("conv_rows: dtype code %d is not known", in_dt);
+#undef KB_CR
+    return check_launch("conv_rows history");
 }
 
 extern "C" int kb_weighted_sum2(float* out, const void* a, int a_dt, int a_splits, long long a_stride, const float* va, const void* b,

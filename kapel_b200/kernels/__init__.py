@@ -383,6 +383,22 @@ def pad_cols(x: torch.Tensor, wide: int) -> torch.Tensor:
     return out
 
 
+def new(shape, dtype: torch.dtype, device) -> torch.Tensor:
+    """Device memory that kernels of several calls fill (each its columns)."""
+    return _fresh(shape, dtype, device)
+
+
+def take_cols(x, off: int, n: int, out_dtype: torch.dtype, wide: int = 0) -> torch.Tensor:
+    """The columns off .. off + n of a product (a tensor or a SplitSum), [rows, n] or `wide` columns with zeros behind."""
+    src, dt, splits, stride = _src(x, "take_cols input")
+    rows, width = x.shape
+    wide = max(int(wide), int(n))
+    out = _fresh((rows, wide), out_dtype, src.device)
+    _check(library().kb_take_cols(_ptr(out), _CODES[out_dtype], _ptr(src), dt, splits, ctypes.c_longlong(stride), int(width), int(off), int(n),
+                                  wide, ctypes.c_longlong(rows), _stream()))
+    return out
+
+
 def gather_rows(x: torch.Tensor, rows: torch.Tensor) -> torch.Tensor:
     _need(x, "gather_rows input", torch.float32)
     _need(rows, "gather_rows rows", torch.int32)
@@ -774,8 +790,8 @@ def paged_attention_mma(q, k_table, v_table, block_table, row_count, tiles, page
     `relative` (decode mode, every tile one token) the multiples are counted from each row's first
     visible key, so a windowed row needs ceil(window / split) slots however long its history. With a
     window, `keep_first` keys from position 0 stay visible below it (prompt portions in one slot only).
-    With `block` > 0 a row at position i sees only the keys from floor(i / block) * block on, and with
-    `sinks` [hq] float32 e^sink joins each row's denominator (both: prompt portions in one slot only)."""
+    With `block` > 0 a row at position i sees only the keys from floor(i / block) * block on (prompt portions
+    in one slot only). With `sinks` [hq] float32 e^sink joins each row's denominator."""
     rows, hq, d = q.shape
     if sinks is not None:
         _need(sinks, "attention sinks", torch.float32, (hq,))
@@ -864,11 +880,13 @@ def proj_norm_append(stacked, q_off: int, k_off: int, v_off: int, q_norm, k_norm
 
 
 def head_gate(y: torch.Tensor, stacked, g_off: int, weight: Optional[torch.Tensor], unit: bool, eps: float,
-              out_dtype: torch.dtype, pad_to: int = 0, gate_act: str = "sigmoid") -> torch.Tensor:
+              out_dtype: torch.dtype, pad_to: int = 0, gate_act: str = "sigmoid", by_head: bool = False, scale: float = 1.0,
+              out: Optional[torch.Tensor] = None, column: int = 0) -> torch.Tensor:
     """y [rows, heads, e] times sigmoid (or, with `gate_act` "silu", silu) of the columns g_off.. of
-    `stacked`; with `unit` each head is first divided by its root mean square (eps inside the
-    root); `weight` [heads e] multiplies too.
-    The result is [rows, heads e], or [rows, pad_to] with zeros behind the heads."""
+    `stacked` (heads e of them, or with `by_head` one a head); with `unit` each head is first divided
+    by its root mean square (eps inside the root); `weight` [heads e] and the number `scale` multiply too.
+    The result is [rows, heads e], or [rows, pad_to] with zeros behind the heads; with `out` [rows, width] the
+    heads go to its columns from `column` on (zeros up to column + pad_to), and it is returned."""
     if gate_act not in GATE_ACTS:
         raise KernelError(f"head_gate: gate activation {gate_act!r} is not known ({sorted(GATE_ACTS)})")
     _need(y, "head_gate input")
@@ -878,12 +896,19 @@ def head_gate(y: torch.Tensor, stacked, g_off: int, weight: Optional[torch.Tenso
         raise KernelError(f"head_gate: {rows} rows against a gate of {g_rows}")
     if weight is not None:
         _need(weight, "head_gate weight", shape=(heads * e,))
-    out_width = max(int(pad_to), heads * e)
-    out = _fresh((rows, out_width), out_dtype, y.device)
+    fill_to = max(int(pad_to), heads * e)
+    if out is None:
+        out, column = _fresh((rows, fill_to), out_dtype, y.device), 0
+    else:
+        _need(out, "head_gate output", out_dtype)
+        if out.dim() != 2 or out.shape[0] != rows or column < 0 or column + fill_to > out.shape[1]:
+            raise KernelError(f"head_gate: columns {column}..{column + fill_to} of an output of {tuple(out.shape)} for {rows} rows")
+    out_width = int(out.shape[1])
+    at = ctypes.c_void_p(out.data_ptr() + int(column) * out.element_size())
     _check(library().kb_head_gate(
-        _ptr(out), _CODES[out_dtype], _ptr(y), _dt(y, "head_gate input"), _ptr(src), dt, splits, ctypes.c_longlong(stride), width,
+        at, _CODES[out_dtype], _ptr(y), _dt(y, "head_gate input"), _ptr(src), dt, splits, ctypes.c_longlong(stride), width,
         int(g_off), _ptr(weight), _dt(weight, "head_gate weight") if weight is not None else F32, int(bool(unit)), _f(eps),
-        ctypes.c_longlong(rows), heads, e, out_width, GATE_ACTS[gate_act], _stream()))
+        ctypes.c_longlong(rows), heads, e, out_width, fill_to, GATE_ACTS[gate_act], int(bool(by_head)), _f(scale), _stream()))
     return out
 
 
@@ -1168,6 +1193,144 @@ def gate_scan(stacked, q_off: int, f_off: int, v_off: int, f_bias: torch.Tensor,
         _ptr(out), _ptr(scratch), _ptr(src), dt, splits, ctypes.c_longlong(stride), width, int(q_off), int(f_off), int(v_off),
         _ptr(f_bias), _ptr(lower), _ptr(state), int(state.shape[0]), _ptr(start), _ptr(end), _ptr(slots), int(entries), rows,
         int(heads), int(d), int(e), _stream()))
+    return out
+
+
+SCAN_MODES = {"gate": 0, "removal": 1, "write": 2, "fixed": 3}      # what the decay scan does to its memory (the kernel file's ScanMode)
+
+
+def _scan_scratch(mode: str, rows: int, heads: int, d: int, e: int, device) -> torch.Tensor:
+    need = int(library().kb_decay_scan_scratch_floats(rows, heads, d, e, SCAN_MODES[mode]))
+    return _fresh((max(1, need),), torch.float32, device)
+
+
+def conv_history_floats(channels: int, taps: int) -> int:
+    """Floats a request keeps between steps for a short convolution over `channels` channels (one that nobody
+    reads where a filter has one weight, so that the state table has a line a request all the same)."""
+    return max(1, (taps - 1) * channels)
+
+
+def _history(state: torch.Tensor, channels: int, taps: int, what: str) -> None:
+    _need(state, f"{what} history", torch.float32)
+    if state.dim() != 2 or state.shape[1] != conv_history_floats(channels, taps):
+        raise KernelError(f"{what}: a history table of {tuple(state.shape)}, expected [slots, {conv_history_floats(channels, taps)}]")
+
+
+def conv_rows(stacked, off: int, channels: int, bias: Optional[torch.Tensor], conv: torch.Tensor, after: Optional[torch.Tensor],
+              state: torch.Tensor, row_entry, ranges, slots, entries: int, taps: int) -> torch.Tensor:
+    """The columns off.. of `stacked` (plus `bias`) through a short causal convolution over time, one filter a
+    channel (`conv` [channels, taps] float32, the last weight for the row itself), plus `after`; float32
+    [rows, channels]. `state` [slots, (taps - 1) channels] holds every request's last inputs."""
+    src, dt, splits, stride, rows, width = _stacked(stacked, "conv_rows input")
+    _need(conv, "conv_rows filters", torch.float32, (channels, taps))
+    for t in (bias, after):
+        if t is not None:
+            _need(t, "conv_rows bias", torch.float32, (channels,))
+    _history(state, channels, taps, "conv_rows")
+    _need(row_entry, "conv_rows row_entry", torch.int32, (rows,))
+    start, end = _ranges(ranges, slots, entries, "conv_rows")
+    out = _fresh((rows, channels), torch.float32, src.device)
+    _check(library().kb_conv_rows(
+        _ptr(out), _ptr(src), dt, splits, ctypes.c_longlong(stride), width, int(off), int(channels), _ptr(bias), _ptr(conv), _ptr(after),
+        _ptr(state), int(state.shape[0]), _ptr(row_entry), _ptr(start), _ptr(end), _ptr(slots), int(entries), rows, int(taps), _stream()))
+    return out
+
+
+def lru_gates(u: torch.Tensor, ra: torch.Tensor, ri: torch.Tensor, ra_bias: torch.Tensor, ri_bias: torch.Tensor, lam: torch.Tensor,
+              rate: float) -> torch.Tensor:
+    """(a, sqrt(1 - a^2) i u) of every row and channel, float32 [rows, width, 2], for u [rows, width] float32 and
+    square matrices `ra`, `ri` [blocks, part, part] over the blocks' channels: a = exp(-rate r softplus(lam)),
+    r = sigmoid(ra u + ra_bias), i = sigmoid(ri u + ri_bias), all in true 32-bit."""
+    _need(u, "lru_gates input", torch.float32)
+    rows, width = u.shape
+    if ra.dim() != 3 or ra.shape[1] != ra.shape[2] or ra.shape[0] * ra.shape[1] != width or tuple(ri.shape) != tuple(ra.shape):
+        raise KernelError(f"lru_gates: matrices of {tuple(ra.shape)} and {tuple(ri.shape)} for {width} channels")
+    _need(ra, "lru_gates recurrence matrices")
+    _need(ri, "lru_gates input matrices", ra.dtype)
+    for t in (ra_bias, ri_bias, lam):
+        _need(t, "lru_gates vectors", torch.float32, (width,))
+    ab = _fresh((rows, width, 2), torch.float32, u.device)
+    _check(library().kb_lru_gates(_ptr(ab), _ptr(u), _ptr(ra), _ptr(ri), _dt(ra, "lru_gates matrices"), _ptr(ra_bias), _ptr(ri_bias), _ptr(lam),
+                                  _f(rate), rows, width, int(ra.shape[0]), _stream()))
+    return ab
+
+
+def lru_scan(ab: torch.Tensor, stacked, y_off: int, y_bias: torch.Tensor, state: torch.Tensor, ranges, slots, entries: int, longest: int,
+             out_dtype: torch.dtype, pad_to: int = 0) -> torch.Tensor:
+    """S <- a S + b over each request's rows, from and into `state` [slots, width], times gelu_tanh of the
+    columns y_off.. of `stacked` plus `y_bias`: [rows, width] (or `pad_to` wide, zeros behind). `longest`: the
+    most rows a request brings (it chooses between walking runs of rows side by side and one thread a channel)."""
+    src, dt, splits, stride, rows, row_width = _stacked(stacked, "lru_scan branch")
+    _need(ab, "lru_scan steps", torch.float32)
+    if ab.dim() != 3 or ab.shape[0] != rows or ab.shape[2] != 2:
+        raise KernelError(f"lru_scan: steps of {tuple(ab.shape)} for {rows} rows")
+    width = int(ab.shape[1])
+    _need(y_bias, "lru_scan bias", torch.float32, (width,))
+    _need(state, "lru_scan state", torch.float32)
+    if state.dim() != 2 or state.shape[1] != width:
+        raise KernelError(f"lru_scan: a state table of {tuple(state.shape)}, expected [slots, {width}]")
+    start, end = _ranges(ranges, slots, entries, "lru_scan")
+    out_width = max(int(pad_to), width)
+    out = _fresh((rows, out_width), out_dtype, src.device)
+    _check(library().kb_lru_scan(
+        _ptr(out), _CODES[out_dtype], out_width, _ptr(ab), _ptr(src), dt, splits, ctypes.c_longlong(stride), row_width, int(y_off), _ptr(y_bias),
+        _ptr(state), int(state.shape[0]), _ptr(start), _ptr(end), _ptr(slots), int(entries), rows, int(longest), width, _stream()))
+    return out
+
+
+def cdelta_scan(stacked, q_off: int, b_off: int, a1_off: int, a2: torch.Tensor, dt_bias: torch.Tensor, a_log: torch.Tensor,
+                conv: torch.Tensor, history: torch.Tensor, memory: torch.Tensor, row_entry, ranges, slots, entries: int, heads: int,
+                kv_heads: int, d: int, e: int, taps: int, q_scale: float, unit_eps: float) -> torch.Tensor:
+    """The read-out [rows, heads, e] (float32, not yet normed) of the gated delta rule with a decay a head and
+    key channel, g = exp(-exp(a_log) softplus(a2 (a1 h) + dt_bias)): S <- diag(g) S; u = beta (v - S^T k);
+    S <- S + k u^T; o = S^T q. The columns q_off.. of `stacked` hold q | k | v (each convolved over `taps` rows,
+    `conv` [2 kv_heads d + heads e, taps], then silu; q and k made unit vectors), b_off.. the step sizes'
+    projections and a1_off.. the decay's first factor. `a2` is its second factor turned, [rank, heads d].
+    `history` [slots, (taps - 1) channels] and `memory` [slots, heads e d] are carried between steps."""
+    src, dt, splits, stride, rows, width = _stacked(stacked, "cdelta input")
+    n, nq, nv = heads * d, kv_heads * d, heads * e
+    channels = 2 * nq + nv
+    _need(a2, "cdelta decay weights", torch.float32)
+    if a2.dim() != 2 or a2.shape[1] != n:
+        raise KernelError(f"cdelta: decay weights of {tuple(a2.shape)}, expected [rank, {n}] (the second factor, turned)")
+    _need(dt_bias, "cdelta decay bias", torch.float32, (n,))
+    _need(a_log, "cdelta decay rates", torch.float32, (heads,))
+    _need(conv, "cdelta filters", torch.float32, (channels, taps))
+    _history(history, channels, taps, "cdelta")
+    _need(memory, "cdelta memory", torch.float32)
+    if memory.dim() != 2 or memory.shape[1] != heads * d * e or memory.shape[0] != history.shape[0]:
+        raise KernelError(f"cdelta: a memory table of {tuple(memory.shape)}, expected [{history.shape[0]}, {heads * d * e}]")
+    _need(row_entry, "cdelta row_entry", torch.int32, (rows,))
+    start, end = _ranges(ranges, slots, entries, "cdelta")
+    out = _fresh((rows, heads, e), torch.float32, src.device)
+    scratch = _scan_scratch("write", rows, heads, d, e, src.device)
+    _check(library().kb_cdelta_scan(
+        _ptr(out), _ptr(scratch), _ptr(src), dt, splits, ctypes.c_longlong(stride), width, int(q_off), int(q_off + nq), int(q_off + 2 * nq),
+        int(b_off), int(a1_off), int(a2.shape[0]), _ptr(a2), _ptr(dt_bias), _ptr(a_log), _ptr(conv), _ptr(history), _ptr(memory),
+        int(memory.shape[0]), _ptr(row_entry), _ptr(start), _ptr(end), _ptr(slots), int(entries), rows, int(heads), int(kv_heads), int(d),
+        int(e), int(taps), _f(q_scale), _f(unit_eps), _stream()))
+    return out
+
+
+def retention_scan(stacked, q_off: int, k_off: int, v_off: int, decay: torch.Tensor, cos_sin, rotary: int, k_scale: float,
+                   state: torch.Tensor, ranges, slots, entries: int, heads: int, d: int, e: int) -> torch.Tensor:
+    """The read-out [rows, heads, e] (float32, not yet normed) of a matrix memory with a fixed decay a head
+    (`decay` [heads]): S <- decay S + k v^T, o = S^T q, queries and keys turned by `cos_sin` [rows, rotary/2, 2]
+    (component i with i + rotary/2), keys then times `k_scale`; `state` [slots, heads e d]."""
+    src, dt, splits, stride, rows, width = _stacked(stacked, "retention input")
+    _need(decay, "retention decays", torch.float32, (heads,))
+    if rotary:
+        _need(cos_sin, "retention cos_sin", torch.float32, (rows, rotary // 2, 2))
+    _need(state, "retention state", torch.float32)
+    if state.dim() != 2 or state.shape[1] != heads * d * e:
+        raise KernelError(f"retention: a state table of {tuple(state.shape)}, expected [slots, {heads * d * e}]")
+    start, end = _ranges(ranges, slots, entries, "retention")
+    out = _fresh((rows, heads, e), torch.float32, src.device)
+    scratch = _scan_scratch("fixed", rows, heads, d, e, src.device)
+    _check(library().kb_retention_scan(
+        _ptr(out), _ptr(scratch), _ptr(src), dt, splits, ctypes.c_longlong(stride), width, int(q_off), int(k_off), int(v_off), _ptr(decay),
+        _ptr(cos_sin if rotary else None), int(rotary), _f(k_scale), _ptr(state), int(state.shape[0]), _ptr(start), _ptr(end), _ptr(slots),
+        int(entries), rows, int(heads), int(d), int(e), _stream()))
     return out
 
 

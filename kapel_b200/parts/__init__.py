@@ -3,6 +3,7 @@ from .attention import Attention
 from .base import (BuildContext, LayerCache, Part, linear, matrix_for, matrix_named, pad_columns, product_width,
                    require_product_widths, stack_rows)
 from .block import ParallelBlock, PostNormBlock, PreNormBlock, SandwichBlock
+from .channel_delta import ChannelDelta
 from .delta import Delta
 from .embedding import Embedding, VocabHead
 from .feed_forward import MLP, GatedMLP
@@ -15,6 +16,8 @@ from .moe import MoE
 from .norm import LayerNorm, RMSNorm, add_branch
 from .parallel import ParallelMixer
 from .position import NoPosition, Rope
+from .retention import Retention
+from .rglru import RGLRU
 from .registry import (
     build_part,
     part_class,
@@ -34,6 +37,9 @@ register_part("mixer", "delta", Delta)
 register_part("mixer", "general_delta", GeneralDelta)
 register_part("mixer", "forget_gate", ForgetGate)
 register_part("mixer", "parallel", ParallelMixer)
+register_part("mixer", "channel_delta", ChannelDelta)
+register_part("mixer", "retention", Retention)
+register_part("mixer", "rglru", RGLRU)
 register_part("merge", "input_mix", InputMix)
 register_part("merge", "input_add", InputAdd)
 register_part("feed_forward", "gated_mlp", GatedMLP)

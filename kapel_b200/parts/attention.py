@@ -13,9 +13,11 @@ kernel that norms q and k and appends k and v to the cache, the row-wise attenti
 knows the kept first keys and the values' size), the gate, the output product.
 
 A spec with an RMS norm over every head's query and key (`q_head_norm`, `k_head_norm`: one weight
-of the head's size for all heads) runs the third path: the stacked product in 32-bit, one kernel
-that norms each head, rotates it and appends keys and values (of their own size) to the cache,
-then the tensor-core kernels where keys and values have one size and the row-wise kernel elsewhere.
+of the head's size for all heads), a sink in the softmax's denominator or one gate a head runs the third
+path: the stacked product in 32-bit, one kernel that norms each head, rotates it and appends keys and
+values (of their own size) to the cache, then the tensor-core kernels where keys and values have one size
+and the row-wise kernel elsewhere, the gate, the output product. A caller that runs two mixers over one
+product may take this path in two steps (`input_names`, `forward_stacked`).
 
 A spec with biases, pooled blocks below the window, a number a head on the scores, mixed heads'
 weights or values mixed with another layer's runs the fourth path (`forward_pooled`): the stacked
@@ -59,7 +61,9 @@ class Attention(Part):
         out = {w["q"]: (qd, spec.hidden), w["k"]: (kvd, spec.hidden), w["v"]: (spec.num_kv_heads * dv, spec.hidden),
                w["o"]: (spec.hidden, spec.num_heads * dv)}
         if spec.gated:
-            out[w["g"]] = (spec.num_heads * dv, spec.hidden)
+            out[w["g"]] = (spec.num_heads if spec.gate_by_head else spec.num_heads * dv, spec.hidden)
+        if spec.sink:
+            out[w["sink"]] = (spec.num_heads,)
         for n in (spec.q_norm, spec.k_norm, spec.q_head_norm, spec.k_head_norm):
             if n is not None:
                 out[n.weight] = (n.width,)
@@ -78,7 +82,9 @@ class Attention(Part):
         if spec.num_heads % spec.num_kv_heads:
             raise ValueError(f"attention: {spec.num_heads} heads over {spec.num_kv_heads} kv heads")
         self.v_dim = spec.v_head_dim or spec.head_dim
-        self.by_head = bool(spec.q_head_norm or spec.k_head_norm)
+        self.by_head = bool(spec.q_head_norm or spec.k_head_norm or spec.sink or spec.gate_by_head)
+        if spec.gate_by_head and not spec.gated:
+            raise ValueError("attention: one gate a head for a layer without a gate")
         self.convolved = bool(spec.conv or spec.values_are_keys or spec.block_mask or spec.unit_sink or spec.qk_bias or spec.out_bias)
         self.out_bias = None
         if self.convolved:
@@ -87,7 +93,7 @@ class Attention(Part):
                                  f"convolutions (1 to 16 rows, got {spec.conv}) whose values are its keys")
             if (self.by_head or spec.gated or spec.q_norm or spec.k_norm or spec.keep_first or spec.softcap or spec.window or spec.bias
                     or spec.pool or spec.head_temp or spec.talk or spec.value_mix or spec.v_head_dim not in (None, spec.head_dim)):
-                raise ValueError("attention: convolutions together with norms, a gate, a window, a soft cap, pooled blocks, mixed heads or "
+                raise ValueError("attention: convolutions together with norms, a sink, a gate, a window, a soft cap, pooled blocks, mixed heads or "
                                  "values of their own are not built")
             if spec.block_mask < 0:
                 raise ValueError(f"attention: blocks of {spec.block_mask} positions")
@@ -95,7 +101,7 @@ class Attention(Part):
         if self.pooled:
             if self.by_head or spec.gated or spec.keep_first or spec.softcap:
                 raise ValueError("attention: biases, pooled blocks, head temperatures, mixed heads or mixed values together with norms "
-                                 "over each head, a gate, kept first keys or a soft cap are not built")
+                                 "over each head, a sink, a gate, kept first keys or a soft cap are not built")
             if spec.pool and (not spec.window or spec.pool_blocks <= 0):
                 raise ValueError(f"attention: blocks of {spec.pool} need a window (got {spec.window}) and a count of blocks (got {spec.pool_blocks})")
             if spec.value_mix not in (None, "source", "mix"):
@@ -103,7 +109,8 @@ class Attention(Part):
         self.general = bool(spec.gated or spec.q_norm or spec.k_norm or spec.keep_first or self.v_dim != spec.head_dim) and not self.by_head \
             and not self.pooled
         if self.by_head and (spec.q_norm or spec.k_norm or spec.keep_first or spec.window):
-            raise ValueError("attention: norms over each head together with norms over the whole projection, a window or kept first keys are not built")
+            raise ValueError("attention: norms over each head, a sink or one gate a head together with norms over the whole projection, a window "
+                             "or kept first keys are not built")
         for n in (spec.q_head_norm, spec.k_head_norm):
             if n is not None and (n.kind != "rms" or n.width != spec.head_dim):
                 raise ValueError(f"attention: a norm over each head must be an RMS norm of width {spec.head_dim}")
@@ -136,6 +143,17 @@ class Attention(Part):
         self.ones = torch.ones((s.hidden,), dtype=torch.float32, device=dev) if s.out_bias else None
         self.sinks = torch.zeros((s.num_heads,), dtype=torch.float32, device=dev) if s.unit_sink else None      # e^0 = 1 in the denominator
 
+    def input_names(self):
+        """The weights whose rows make up the stacked product, in order; None where the layer cannot share one."""
+        w = self.spec.weights
+        return [w["q"], w["k"], w["v"]] + ([w["g"]] if self.spec.gated else []) if self.by_head else None
+
+    def load_shared(self, tensors):
+        """`load` without the two products' weights, for a caller that multiplies by them (`forward_stacked`)."""
+        s = self.spec
+        self.sinks = tensors[s.weights["sink"]].to(self.ctx.device).float().contiguous() if s.sink else None
+        self.load_norms(tensors)
+
     def load(self, tensors):
         if self.convolved:
             return self.load_convolved(tensors)
@@ -143,7 +161,10 @@ class Attention(Part):
         names = [w["q"], w["k"], w["v"]] + ([w["g"]] if self.spec.gated else [])
         self.w_qkv = stack_rows(self.ctx, tensors, names, "attention")
         self.w_o = matrix_named(self.ctx, tensors, w["o"])
-        if (self.general and self.spec.gated) or self.by_head or self.pooled:
+        if self.by_head:
+            self.w_o = pad_columns(self.ctx, self.w_o)
+            return self.load_shared(tensors)
+        if (self.general and self.spec.gated) or self.pooled:
             self.w_o = pad_columns(self.ctx, self.w_o)
         if self.pooled:
             dev = self.ctx.device
@@ -152,6 +173,9 @@ class Attention(Part):
             self.temp = tensors[w["temp"]].to(dev).float().contiguous() if self.spec.head_temp else None
             self.talk = tensors[w["talk"]].to(dev).float().contiguous() if self.spec.talk else None
             self.v_weight = small(w["vmix"]).reshape(1) if self.spec.value_mix == "mix" else None
+        self.load_norms(tensors)
+
+    def load_norms(self, tensors):
         self.proj_norms = []
         for n in (self.spec.q_head_norm, self.spec.k_head_norm) if self.by_head else (self.spec.q_norm, self.spec.k_norm):
             if n is None:
@@ -273,33 +297,40 @@ class Attention(Part):
         return linear(self.ctx, y.view(y.shape[0], s.num_heads * dv), self.w_o, keep_split=True)
 
     def forward_by_head(self, h, batch, cache):
+        stacked = linear(self.ctx, h, self.w_qkv, out_dtype=torch.float32, keep_split=True)
+        return linear(self.ctx, self.forward_stacked(stacked, 0, batch, cache), self.w_o, keep_split=True)
+
+    @property
+    def inner_width(self) -> int:
+        return self.spec.num_heads * self.v_dim
+
+    def forward_stacked(self, stacked, base: int, batch, cache, out=None, column: int = 0, pad_to=None, scale: float = 1.0):
+        """The output product's input [rows, heads x value size] (padded to the product's width), from the columns
+        `base`.. of a stacked product; with `out`, times `scale` and written to its columns from `column` on, zeros
+        up to `column` + `pad_to`."""
         s, dv = self.spec, self.v_dim
         nq, nk = s.num_heads * s.head_dim, s.num_kv_heads * s.head_dim
-        stacked = linear(self.ctx, h, self.w_qkv, out_dtype=torch.float32, keep_split=True)
         k_table, v_table = cache.tables()
         group = batch.groups[cache.group]
         rotary = self.position.rotary_dim
-        q = K.head_norm_rope_append(stacked, 0, nq, nq + nk, self.proj_norms[0], self.proj_norms[1],
+        q = K.head_norm_rope_append(stacked, base, base + nq, base + nq + nk, self.proj_norms[0], self.proj_norms[1],
                                     self.position.tables(batch) if rotary else None, rotary, group.lines, k_table, v_table,
                                     s.num_heads, s.num_kv_heads, s.head_dim, dv, cache.owns, self.ctx.dtype)
         heads_per_kv = s.num_heads // s.num_kv_heads
         if dv == s.head_dim and s.head_dim % 16 == 0 and K.attention_mma_takes(q.dtype, s.head_dim, heads_per_kv):
-            decode, tiles, split, slots, relative = batch.attention_tiles(
-                heads_per_kv, s.num_kv_heads, None, s.head_dim,
-                K.attention_prompt_kernel(s.num_heads, s.num_kv_heads, s.head_dim, self.ctx.page_size, s.softcap))
+            prompt = "mma" if self.sinks is not None else K.attention_prompt_kernel(s.num_heads, s.num_kv_heads, s.head_dim, self.ctx.page_size, s.softcap)
+            decode, tiles, split, slots, relative = batch.attention_tiles(heads_per_kv, s.num_kv_heads, None, s.head_dim, prompt)
             y = K.paged_attention_mma(q, k_table, v_table, group.block_table, batch.row_count, tiles, self.ctx.page_size, None,
-                                      s.scale, s.softcap, decode, split, slots, relative, pairs=getattr(batch, "pairs", None))
+                                      s.scale, s.softcap, decode, split, slots, relative, pairs=getattr(batch, "pairs", None), sinks=self.sinks)
         else:
             y = K.paged_attention_rows(q, k_table, v_table, group.block_table, batch.row_entry, batch.row_count, self.ctx.page_size,
-                                       None, s.scale, s.softcap, batch.attention_slots(None))
-        width = product_width(self.ctx, s.num_heads * dv)
-        if s.gated:
-            y = K.head_gate(y, stacked, nq + nk + s.num_kv_heads * dv, None, False, 0.0, self.ctx.dtype, pad_to=width)
-        else:
-            y = y.view(y.shape[0], s.num_heads * dv)
-            if width != y.shape[1]:
-                y = K.pad_cols(y, width)
-        return linear(self.ctx, y, self.w_o, keep_split=True)
+                                       None, s.scale, s.softcap, batch.attention_slots(None), sinks=self.sinks)
+        width = product_width(self.ctx, s.num_heads * dv) if pad_to is None else pad_to
+        if s.gated or out is not None:
+            return K.head_gate(y, stacked, base + nq + nk + s.num_kv_heads * dv if s.gated else 0, None, False, 0.0, self.ctx.dtype, pad_to=width,
+                               gate_act="sigmoid" if s.gated else "none", by_head=s.gate_by_head, scale=scale, out=out, column=column)
+        y = y.view(y.shape[0], s.num_heads * dv)
+        return K.pad_cols(y, width) if width != y.shape[1] else y
 
     def forward(self, h, batch, cache):
         s = self.spec

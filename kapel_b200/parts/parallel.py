@@ -1,8 +1,11 @@
 """Two mixers side by side that read the same input: left_scale * left(h) + right_scale * right(h).
 
 Each side keeps what it keeps under its own name in the layer's cache (`CacheNeeds.named`), and sees
-the cache through that name (`LayerCache.scoped`); at most one side asks for pages. The weighted sum
-is one kernel in 32-bit; a side whose output product has a bias that it can leave to its caller
+the cache through that name (`LayerCache.scoped`); at most one side asks for pages. Where both sides can
+take their inputs from a product made for both (`input_names`, `forward_stacked`), the layer is one stacked
+product for all roles of both sides, the sides' own steps, which leave their scaled results side by side in
+one row, and one output product over both. Elsewhere each side runs its own products and the weighted sum is
+one kernel in 32-bit; a side whose output product has a bias that it can leave to its caller
 (`forward_unbiased` and `out_bias`) has it added there.
 """
 from __future__ import annotations
@@ -10,7 +13,7 @@ from __future__ import annotations
 import torch
 
 from .. import kernels as K
-from .base import Part
+from .base import Part, linear, matrix_for, pad_columns, stack_rows
 from .registry import build_part, part_class
 
 
@@ -26,13 +29,26 @@ class ParallelMixer(Part):
         super().__init__(spec, ctx)
         self.left = build_part("mixer", spec.left, ctx)
         self.right = build_part("mixer", spec.right, ctx)
+        names = [side.input_names() if hasattr(side, "input_names") else None for side in (self.left, self.right)]
+        self.names = names if all(n is not None for n in names) else None      # one product for both sides
         self.cache_needs()                      # refuses two sides that both want pages
 
     @property
     def graph_safe(self) -> bool:
         return self.left.graph_safe and self.right.graph_safe
 
+    def load_shared(self, tensors):
+        expected = self.expected_tensors(self.spec)
+        self.w_in = stack_rows(self.ctx, tensors, self.names[0] + self.names[1], "parallel")
+        self.right_base = sum(expected[n][0] for n in self.names[0])
+        out = [matrix_for(self.ctx, tensors[side.weights["o"]]) for side in (self.spec.left, self.spec.right)]
+        self.w_o = pad_columns(self.ctx, torch.cat(out, dim=1).contiguous())
+        self.left.load_shared(tensors)
+        self.right.load_shared(tensors)
+
     def load(self, tensors):
+        if self.names is not None:
+            return self.load_shared(tensors)
         self.left.load(tensors)
         self.right.load(tensors)
         s, dev = self.spec, self.ctx.device
@@ -50,6 +66,17 @@ class ParallelMixer(Part):
     def cache_needs(self):
         return self.left.cache_needs().named("left").merged(self.right.cache_needs().named("right"))
 
+    def forward_shared(self, h, batch, cache):
+        s, split = self.spec, self.left.inner_width
+        stacked = linear(self.ctx, h, self.w_in, out_dtype=torch.float32, keep_split=True)
+        both = K.new((h.shape[0], self.w_o.shape[1]), self.ctx.dtype, h.device)
+        self.left.forward_stacked(stacked, 0, batch, cache.scoped("left"), out=both, column=0, pad_to=split, scale=s.left_scale)
+        self.right.forward_stacked(stacked, self.right_base, batch, cache.scoped("right"), out=both, column=split,
+                                   pad_to=self.w_o.shape[1] - split, scale=s.right_scale)
+        return linear(self.ctx, both, self.w_o, keep_split=True)
+
     def forward(self, h, batch, cache):
+        if self.names is not None:
+            return self.forward_shared(h, batch, cache)
         run = lambda side, name: (side.forward_unbiased if hasattr(side, "forward_unbiased") else side.forward)(h, batch, cache.scoped(name))
         return K.weighted_sum2(run(self.left, "left"), self.va, run(self.right, "right"), self.vb, self.vc)

@@ -14,15 +14,28 @@ import math
 import torch
 
 from .. import kernels as K
+from ..config.spec import RopeBands
 from .base import Part
 
 
+def _banded(f: float, b: RopeBands) -> float:
+    turns = b.original * f / (2.0 * math.pi)                # original / wavelength: how often the pair turns over `original` positions
+    if turns >= b.high:
+        return f
+    if turns <= b.low:
+        return f / b.factor
+    s = (turns - b.low) / (b.high - b.low)
+    return (1.0 - s) * f / b.factor + s * f
+
+
 def scaled_frequencies(rotary_dim: int, theta: float, scaling):
-    """(frequency of every pair as a list of floats, the factor on cos and sin) for `spec.RopeScaling`."""
+    """(frequency of every pair as a list of floats, the factor on cos and sin) for `spec.RopeScaling` or `spec.RopeBands`."""
     half = rotary_dim // 2
     f = [theta ** (-2.0 * j / rotary_dim) for j in range(half)]
     if scaling is None:
         return f, 1.0
+    if isinstance(scaling, RopeBands):
+        return [_banded(x, scaling) for x in f], 1.0
 
     def pair_of(turns: float) -> float:
         return rotary_dim * math.log(scaling.original / (2.0 * math.pi * turns)) / (2.0 * math.log(theta))
@@ -44,7 +57,10 @@ class Rope(Part):
         if spec.pairing not in ("half", "neighbours"):
             raise ValueError(f"rope pairing {spec.pairing!r} is not built (\"half\", \"neighbours\")")
         scaling = getattr(spec, "scaling", None)
-        if scaling is not None and not (scaling.factor > 0 and scaling.original > 0 and scaling.fast > 0 and scaling.slow > 0 and spec.theta > 1):
+        if isinstance(scaling, RopeBands):
+            if not (scaling.factor > 0 and scaling.original > 0 and scaling.high >= scaling.low > 0):
+                raise ValueError(f"rope scaling {scaling} needs positive numbers and a high bound that is not below the low one")
+        elif scaling is not None and not (scaling.factor > 0 and scaling.original > 0 and scaling.fast > 0 and scaling.slow > 0 and spec.theta > 1):
             raise ValueError(f"rope scaling {scaling} needs positive numbers and a base above 1")
         self._freqs = None
         if scaling is not None:                             # made when the part is built: a recorded step reads the same device tensor again
