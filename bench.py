@@ -1,7 +1,7 @@
 """Throughput of the engine at Gemma 2 sizes with random weights, on one GPU.
 
     python bench.py [--gpus 1] [--steps K] [--warmup W] [--size 2b|9b|27b] [--layers L] [--impl reference]
-    python bench.py --design fusitar|kofutar|teluzen|lokedra [--design-sizes s,m]      (another line: see `design_line`)
+    python bench.py --design fusitar|kofutar|teluzen|lokedra|mukunex [--design-sizes s,m]      (another line: see `design_line`)
 
 A "step" is one decode step. The default run has the layer sizes of the 2B configuration
 (26 layers, hidden 2304, 8 heads over 4 kv heads of 256, intermediate 9216, vocabulary 256000,
@@ -451,6 +451,28 @@ def lokedra_config(z):
             "layers": [(par, rec, lat, rec)[i % 4] for i in range(z["layers"])]}
 
 
+# --design mukunex: the Mukunex design (attention with a sink and a gate a head beside retention, over one product; a
+# real-gated linear recurrent unit; the delta rule with a decay a channel; dense gated feed-forwards) beside Kofutar, the
+# engine's other design with causal attention on the same kernels, a delta rule and dense feed-forwards, and Lokedra, its
+# other design with two mixers side by side, linear attention and the decay scan, at equal sizes: the same width, heads, head
+# size, vocabulary, as many layers, Kofutar's feed-forward. Its layers take turns: parallel, unit, parallel, delta; the unit
+# is as wide as the model in parts of a head's size; the low ranks are Lokedra's.
+def mukunex_config(z):
+    mlp = {"kind": "dense", "ff": z["top"] * z["ff"]}
+    bands = {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 1024}
+    par = {"type": "parallel", "mlp": mlp, "mixer": {
+        "left": {"heads": z["heads"], "kv_heads": z["kv_heads"], "dim": z["dim"], "vdim": z["dim"], "scale": z["dim"] ** -0.5,
+                 "rot": {"base": 10000.0, "dims": z["dim"], "scaling": bands}},
+        "right": {"heads": z["heads"], "dim": z["dim"], "vdim": z["dim"], "decay": [1.0 - 2.0 ** -(5 + i % 8) for i in range(z["heads"])],
+                  "rot": {"base": 10000.0, "dims": z["dim"]}},
+        "left_scale": 1.0, "right_scale": 1.0}}
+    lru = {"type": "rglru", "mlp": mlp, "mixer": {"width": z["width"], "blocks": z["width"] // z["dim"], "conv": 4}}
+    rec = {"type": "channel_delta", "mlp": mlp, "mixer": {"heads": z["heads"], "kv_heads": z["kv_heads"], "dim": z["dim"], "vdim": z["dim"],
+                                                            "conv": 4, "decay_rank": LOKEDRA_LORA, "gate_rank": LOKEDRA_LORA}}
+    return {"architecture": "Mukunex", "vocab": z["vocab"], "width": z["width"], "norm": {"eps": 1e-6},
+            "layers": [(par, lru, par, rec)[i % 4] for i in range(z["layers"])]}
+
+
 def gemma_config(z):
     return {"architectures": ["Gemma2ForCausalLM"], "model_type": "gemma2", "num_hidden_layers": z["layers"], "hidden_size": z["width"],
             "num_attention_heads": z["heads"], "num_key_value_heads": z["kv_heads"], "head_dim": z["dim"],
@@ -476,6 +498,20 @@ def design_kernel_rooflines(which, z, kind, rows, context, batch, pk):
         experts_read = min(z["experts"], batch * (z["top"] - 1)) + 1
         return {"attention": ("bytes", layers * batch * (min(context, win) * hkv * 2 * d * 2.0 + (max(0, context - win) // TELUZEN_POOL) * hkv * 2 * d * 4.0)),
                 "feed_forward": ("bytes", 2.0 * z["top"] * z["ff"] * w * 2 + moe_layers * experts_read * 3.0 * z["ff"] * w * 2)}
+    if which == "mukunex":
+        par_layers, lru_layers, rec_layers = (layers + 1) // 2, (layers + 2) // 4, layers // 4
+        ff = z["top"] * z["ff"]
+        if kind == "prefill":
+            pairs = rows * (rows + 1) // 2
+            # a row and head: retention decays and writes (3 a value of the [d, d] memory) and reads once (2); the delta rule
+            # decays, writes (3) and reads twice (4). The unit's kernels move both branches in 32-bit in and the product's input out.
+            return {"attention": ("flops", par_layers * 4.0 * pairs * hq * d), "feed_forward": ("flops", layers * 2.0 * rows * 3 * ff * w),
+                    "retention_scan": ("flops", par_layers * 5.0 * rows * hq * d * d), "delta_scan": ("flops", rec_layers * 7.0 * rows * hq * d * d),
+                    "recurrent_unit": ("bytes", lru_layers * rows * w * (4 + 4 + 2.0))}
+        state = batch * hq * d * d * 4 * 2.0
+        return {"attention": ("bytes", par_layers * batch * context * hkv * d * 2 * 2.0), "feed_forward": ("bytes", layers * 3.0 * ff * w * 2),
+                "retention_scan": ("bytes", par_layers * state), "delta_scan": ("bytes", rec_layers * state),
+                "recurrent_unit": ("bytes", lru_layers * (2.0 * w * d * 2 + batch * w * (4 + 4 + 2 + 4 * 2 * 4.0)))}
     if which == "lokedra":
         par_layers, lat_layers, rec_layers = (layers + 3) // 4, (layers + 1) // 4, layers // 2
         r, kv = 64, KOFUTAR_KV_RANK
@@ -553,6 +589,17 @@ LOKEDRA_KERNEL_CLASSES = {
 }
 
 
+# Mukunex's attention and feed-forwards run the kernels Kofutar's run; its two memories the decay scan behind their own inputs'
+# kernels; the recurrent unit has the convolution, the gates' products and the scan of one number a channel.
+MUKUNEX_KERNEL_CLASSES = {
+    "attention": ("paged_attention_mma", "paged_attention_rows"),
+    "feed_forward": ("gemm_glu_fused", "glu"),
+    "retention_scan": ("retention_scan",),
+    "delta_scan": ("cdelta_scan",),
+    "recurrent_unit": ("conv_rows", "lru_gates", "lru_scan"),
+}
+
+
 def design_point(which, z, steps, warmup, clocks, pk):
     """Prefill of 2,048 tokens and decode at batch 8 for one design at one size: tokens a second through
     the engine (recorded passes), and the device time of each kernel entry point in one eager pass."""
@@ -562,7 +609,8 @@ def design_point(which, z, steps, warmup, clocks, pk):
     from kapel_b200 import kernels as K
     from kapel_b200.engine import Engine, StepEntry
 
-    cfg = {"fusitar": fusitar_config, "kofutar": kofutar_config, "gemma2": gemma_config, "teluzen": teluzen_config, "lokedra": lokedra_config}[which](z)
+    cfg = {"fusitar": fusitar_config, "kofutar": kofutar_config, "gemma2": gemma_config, "teluzen": teluzen_config, "lokedra": lokedra_config,
+           "mukunex": mukunex_config}[which](z)
     room = (DESIGN_BATCH + 1) * (DESIGN_HISTORY + 4 * (steps + warmup) + 128) + PREFILL_TOKENS
     engine = Engine.random(cfg, seed=0, dtype="bfloat16", max_tokens=room, max_sequences=DESIGN_BATCH + 2)
     rng = np.random.default_rng(0)
@@ -607,18 +655,22 @@ def design_point(which, z, steps, warmup, clocks, pk):
         must = design_kernel_rooflines(which, z, kind, PREFILL_TOKENS, DESIGN_HISTORY, DESIGN_BATCH, pk)
         classes = {}
         for name, shape, calls, ms in rows:
-            for cls, members in {"kofutar": KOFUTAR_KERNEL_CLASSES, "teluzen": TELUZEN_KERNEL_CLASSES, "lokedra": LOKEDRA_KERNEL_CLASSES}.get(which, KERNEL_CLASSES).items():
+            for cls, members in {"kofutar": KOFUTAR_KERNEL_CLASSES, "teluzen": TELUZEN_KERNEL_CLASSES, "lokedra": LOKEDRA_KERNEL_CLASSES,
+                                 "mukunex": MUKUNEX_KERNEL_CLASSES}.get(which, KERNEL_CLASSES).items():
                 if name in members:
                     classes[cls] = classes.get(cls, 0.0) + ms
-        if which in ("gemma2", "kofutar"):   # the dense way down is a plain product: count the products whose inner width is the intermediate size
+        if which in ("gemma2", "kofutar", "mukunex"):   # the dense way down is a plain product: count the products whose inner width is the intermediate size
             # (Kofutar's input mix has the same shape where the intermediate size is twice the width: one call more than the layers', taken off by its share)
             classes["feed_forward"] = classes.get("feed_forward", 0.0) + sum(
                 ms * (z["layers"] / calls if (which == "kofutar" and calls == z["layers"] + 1) else 1.0)
                 for name, shape, calls, ms in rows if name == "gemm" and len(shape) == 2 and shape[0] == z["width"] and shape[1] == z["top"] * z["ff"])
+        if which == "mukunex":             # a parallel layer's output product, over both sides' results, may have the way down's shape: off by its share
+            classes["feed_forward"] -= sum(ms * (1.0 - z["layers"] / calls) for name, shape, calls, ms in rows
+                                           if name == "gemm" and len(shape) == 2 and shape[0] == z["width"] and shape[1] == z["top"] * z["ff"] and calls > z["layers"])
         if which == "teluzen":             # the ways down of the plain layer and of the shared expert
             classes["feed_forward"] = classes.get("feed_forward", 0.0) + sum(
                 ms for name, shape, calls, ms in rows if name == "gemm" and len(shape) == 2 and shape[0] == z["width"] and shape[1] in (z["ff"], z["top"] * z["ff"]))
-        rec = {"kernels": [{"name": n, "shape": list(sh), "calls": c, "ms": round(ms, 4)} for n, sh, c, ms in rows][:14], "classes": {}}
+        rec = {"kernels": [{"name": n, "shape": list(sh), "calls": c, "ms": round(ms, 4)} for n, sh, c, ms in rows][:24], "classes": {}}
         for cls, ms in classes.items():
             unit, amount = must[cls]
             if amount <= 0 or ms <= 0:
@@ -645,7 +697,7 @@ def design_line(args) -> int:
     sizes = {}
     for name in args.design_sizes.split(","):
         z = DESIGN_SIZES[name]
-        beside = ("gemma2",) if args.design == "fusitar" else (("kofutar", "fusitar") if args.design == "lokedra" else ("fusitar", "gemma2"))
+        beside = {"fusitar": ("gemma2",), "lokedra": ("kofutar", "fusitar"), "mukunex": ("kofutar", "lokedra")}.get(args.design, ("fusitar", "gemma2"))
         if args.design_beside is not None:
             beside = tuple(b for b in args.design_beside.split(",") if b)
         sizes[name] = {"shape": z}
@@ -677,8 +729,8 @@ def main() -> int:
     ap.add_argument("--skip-check", action="store_true", help="leave out the check of the timed logits against the 32-bit path")
     ap.add_argument("--breakdown", action="store_true",
                     help="instead of the JSON line: device time by kernel for one prefill step and one eager decode step")
-    ap.add_argument("--design", default=None, choices=["fusitar", "kofutar", "teluzen", "lokedra"],
-                    help="instead of the default line: this design beside Gemma 2 (kofutar and teluzen: beside Fusitar and Gemma 2; lokedra: beside Kofutar and Fusitar) at equal sizes, prefill and decode, with each like kernel's roofline fraction")
+    ap.add_argument("--design", default=None, choices=["fusitar", "kofutar", "teluzen", "lokedra", "mukunex"],
+                    help="instead of the default line: this design beside Gemma 2 (kofutar and teluzen: beside Fusitar and Gemma 2; lokedra: beside Kofutar and Fusitar; mukunex: beside Kofutar and Lokedra) at equal sizes, prefill and decode, with each like kernel's roofline fraction")
     ap.add_argument("--design-beside", default=None, help="which other designs run beside it (comma separated; empty: none); default: the closest ones")
     ap.add_argument("--design-sizes", default="s,m", help="which of the design sizes (s, m), comma separated")
     args = ap.parse_args()

@@ -6,12 +6,14 @@
 // S is one float a channel in a slot of a state table, one slot a request, carried from a request's last
 // row in this step to its first row in the next. Everything here is 32-bit.
 //
-// Two kernels. The gates' kernel makes (a, sqrt(1 - a^2) i u) of every row and channel: two square products
-// a part, taken in true 32-bit (tiles of 64 rows by 32 channels; for a few rows a warp a channel). The scan's
-// kernel walks a request's rows: a step x -> a x + b composes ((a1, b1) then (a2, b2) is (a1 a2, a2 b1 + b2)),
-// so a block takes 16 channels and 32 runs of 8 rows at a time, each thread composing one run, the runs joined
-// by a scan over a warp's lanes; then every thread walks its rows again from the state before them. A step
-// of few rows a request is walked by one thread a channel.
+// Two kernels. The gates' kernel makes (a - 1, sqrt(1 - a^2) i u) of every row and channel: two square products
+// a part, taken in true 32-bit (tiles of 64 rows by 32 channels; for a few rows a warp a channel). A memory of
+// thousands of rows has decays so near 1 that rounding a itself would be most of the error: a - 1 keeps its own
+// precision, and a row is S <- S + ((a - 1) S + b), rounded once. The scan's kernel walks a request's rows: a
+// step composes ((x1, b1) then (x2, b2) is (x1 + x2 + x1 x2, b1 + x2 b1 + b2) with x = a - 1), so a block takes
+// 16 channels and 32 runs of 8 rows at a time, each thread composing one run, the runs joined by a scan over a
+// warp's lanes; then every thread walks its rows again from the state before them. A step of few rows a request
+// is walked by one thread a channel.
 #include "common.cuh"
 
 namespace kb {
@@ -23,7 +25,7 @@ struct LruGateParams {
     const float* ra_bias;       // [width]
     const float* ri_bias;
     const float* lam;           // [width]
-    float2* ab;                 // [rows, width]: (a, what is added)
+    float2* ab;                 // [rows, width]: (a - 1, what is added)
     float rate;
     int rows, width, part;      // part = width / blocks
 };
@@ -34,8 +36,12 @@ __device__ __forceinline__ float2 lru_step(const LruGateParams& p, int c, float 
     const float lam = p.lam[c];
     const float sp = lam > 20.f ? lam : log1pf(expf(lam));
     const float log_a = -p.rate * lru_sigmoid(zr + p.ra_bias[c]) * sp;
-    return make_float2(expf(log_a), sqrtf(-expm1f(2.f * log_a)) * lru_sigmoid(zi + p.ri_bias[c]) * u);
+    const float x = expm1f(log_a);                              // a - 1; 1 - a^2 = -x (x + 2)
+    return make_float2(x, sqrtf(-x * (x + 2.f)) * lru_sigmoid(zi + p.ri_bias[c]) * u);
 }
+
+// A step (x, b) on a state, and on what an earlier step does (b1; its x1 likewise with b = x).
+__device__ __forceinline__ float lru_apply(float x, float b, float S) { return S + fmaf(x, S, b); }
 
 constexpr int LG_ROWS = 64, LG_COLS = 32, LG_K = 32, LG_THREADS = 256;
 
@@ -169,7 +175,7 @@ lru_scan_kernel(const Src<TS> src, const LruScanParams p, TO* __restrict__ out) 
 #pragma unroll
         for (int j = 0; j < LS_ROWS; ++j) {
             const int r = base + s * LS_ROWS + j;
-            next[j] = (mine && r < r1) ? p.ab[(size_t)r * p.width + c] : make_float2(1.f, 0.f);
+            next[j] = (mine && r < r1) ? p.ab[(size_t)r * p.width + c] : make_float2(0.f, 0.f);
         }
     };
     fetch(r0);
@@ -183,26 +189,26 @@ lru_scan_kernel(const Src<TS> src, const LruScanParams p, TO* __restrict__ out) 
             y[j] = (mine && r < r1) ? src.at((size_t)r * p.row_width + p.y_off + c) : 0.f;
         }
         if (base + LS_RUNS * LS_ROWS < r1) fetch(base + LS_RUNS * LS_ROWS);
-        float A = 1.f, B = 0.f;
+        float X = 0.f, B = 0.f;
 #pragma unroll
         for (int j = 0; j < LS_ROWS; ++j) {
-            A *= ab[j].x;
-            B = fmaf(ab[j].x, B, ab[j].y);
+            X = lru_apply(ab[j].x, ab[j].x, X);
+            B = lru_apply(ab[j].x, ab[j].y, B);
         }
-        run[s][cl] = make_float2(A, B);
+        run[s][cl] = make_float2(X, B);
         __syncthreads();
         {                                                       // warp w joins the runs of channel w, lane l being run l
             float2 f = run[lane][warp];
 #pragma unroll
             for (int o = 1; o < 32; o <<= 1) {
-                const float a1 = __shfl_up_sync(0xffffffffu, f.x, o), b1 = __shfl_up_sync(0xffffffffu, f.y, o);
-                if (lane >= o) {                                // f after (a1, b1)
-                    f.y = fmaf(f.x, b1, f.y);
-                    f.x *= a1;
+                const float x1 = __shfl_up_sync(0xffffffffu, f.x, o), b1 = __shfl_up_sync(0xffffffffu, f.y, o);
+                if (lane >= o) {                                // f after (x1, b1)
+                    f.y = lru_apply(f.x, f.y, b1);
+                    f.x = lru_apply(f.x, f.x, x1);
                 }
             }
             const float start = carry[warp];
-            const float after = fmaf(f.x, start, f.y);          // the state behind this lane's run
+            const float after = lru_apply(f.x, f.y, start);          // the state behind this lane's run
             float before = __shfl_up_sync(0xffffffffu, after, 1);
             if (lane == 0) before = start;
             __syncwarp();
@@ -214,7 +220,7 @@ lru_scan_kernel(const Src<TS> src, const LruScanParams p, TO* __restrict__ out) 
 #pragma unroll
         for (int j = 0; j < LS_ROWS; ++j) {
             const int r = base + s * LS_ROWS + j;
-            S = fmaf(ab[j].x, S, ab[j].y);
+            S = lru_apply(ab[j].x, ab[j].y, S);
             if (mine && r < r1) Elem<TO>::store(out + (size_t)r * p.out_stride + c, S * gelu_tanh(y[j] + bias));
         }
         __syncthreads();                                        // the runs may be written again
@@ -237,7 +243,7 @@ __global__ void lru_scan_few_kernel(const Src<TS> src, const LruScanParams p, TO
         float o = 0.f;
         if (live) {
             const float2 ab = p.ab[(size_t)r * p.width + c];
-            S = fmaf(ab.x, S, ab.y);
+            S = lru_apply(ab.x, ab.y, S);
             o = S * gelu_tanh(src.at((size_t)r * p.row_width + p.y_off + c) + bias);
         }
         Elem<TO>::store(out + (size_t)r * p.out_stride + c, o);
@@ -249,7 +255,7 @@ __global__ void lru_scan_few_kernel(const Src<TS> src, const LruScanParams p, TO
 
 using namespace kb;
 
-// ab [rows, width, 2] = (a, sqrt(1 - a^2) i u) of every row and channel.
+// ab [rows, width, 2] = (a - 1, sqrt(1 - a^2) i u) of every row and channel.
 extern "C" int kb_lru_gates(float* ab, const float* u, const void* ra, const void* ri, int w_dt, const float* ra_bias, const float* ri_bias,
                             const float* lam, float rate, int rows, int width, int blocks, void* stream) {
     KB_REQUIRE(rows >= 0 && width > 0 && blocks > 0 && width % blocks == 0, "lru_gates: rows %d, %d channels in %d parts", rows, width, blocks);

@@ -1238,7 +1238,7 @@ def conv_rows(stacked, off: int, channels: int, bias: Optional[torch.Tensor], co
 
 def lru_gates(u: torch.Tensor, ra: torch.Tensor, ri: torch.Tensor, ra_bias: torch.Tensor, ri_bias: torch.Tensor, lam: torch.Tensor,
               rate: float) -> torch.Tensor:
-    """(a, sqrt(1 - a^2) i u) of every row and channel, float32 [rows, width, 2], for u [rows, width] float32 and
+    """(a - 1, sqrt(1 - a^2) i u) of every row and channel, float32 [rows, width, 2], for u [rows, width] float32 and
     square matrices `ra`, `ri` [blocks, part, part] over the blocks' channels: a = exp(-rate r softplus(lam)),
     r = sigmoid(ra u + ra_bias), i = sigmoid(ri u + ri_bias), all in true 32-bit."""
     _need(u, "lru_gates input", torch.float32)
@@ -1257,7 +1257,7 @@ def lru_gates(u: torch.Tensor, ra: torch.Tensor, ri: torch.Tensor, ra_bias: torc
 
 def lru_scan(ab: torch.Tensor, stacked, y_off: int, y_bias: torch.Tensor, state: torch.Tensor, ranges, slots, entries: int, longest: int,
              out_dtype: torch.dtype, pad_to: int = 0) -> torch.Tensor:
-    """S <- a S + b over each request's rows, from and into `state` [slots, width], times gelu_tanh of the
+    """S <- a S + b over each request's rows (`ab` holds a - 1 and b), from and into `state` [slots, width], times gelu_tanh of the
     columns y_off.. of `stacked` plus `y_bias`: [rows, width] (or `pad_to` wide, zeros behind). `longest`: the
     most rows a request brings (it chooses between walking runs of rows side by side and one thread a channel)."""
     src, dt, splits, stride, rows, row_width = _stacked(stacked, "lru_scan branch")
@@ -1689,7 +1689,7 @@ _TIMED = ("embed", "rope_table", "rope_append", "glu", "cast", "gather_rows", "r
           "moe_sort", "moe_grouped", "moe_combine", "gemm_glu_fused", "paged_attention_decode_fused", "layernorm", "concat2",
           "head_norm_rope_append", "latent_append", "head_linear", "delta_scan", "latent_attention_mma", "proj_rope_append",
           "pool_blocks", "pooled_attention", "act", "token_shift", "conv_append", "gdelta_scan", "gate_scan", "weighted_sum2",
-          "glu_clamped")
+          "glu_clamped", "cdelta_scan", "retention_scan", "conv_rows", "lru_gates", "lru_scan", "take_cols")
 _timing = None
 _originals = {}
 
