@@ -26,6 +26,12 @@
 
 namespace kb {
 
+// retention.cu: a fixed decay's memory by chunks of rows
+long long retention_chunk_floats(int rows, int entries, int heads, int d, int e);
+int run_retention_chunks(float* out, const float* vec, const float* val, const float* scal, const float* decay, float* sums, float* state,
+                         int n_slots, const int* entry_start, const int* entry_end, const int* slots, int entries, int longest, int heads,
+                         int d, int e, cudaStream_t s);
+
 typedef __nv_bfloat16 bf16;
 
 __device__ __forceinline__ float rc_sigmoid(float x) { return 1.f / (1.f + expf(-x)); }
@@ -940,11 +946,22 @@ extern "C" int kb_cdelta_scan(float* out, float* scratch, const void* src, int i
     return run_decay_scan(out, in, memory, n_slots, entry_start, entry_end, slots, entries, heads, d, e, SCAN_WRITE, nullptr, s);
 }
 
-// The read-out [rows, heads, e] of a matrix memory with a fixed decay a head behind rotated queries and keys.
+// From how many rows of a request on the memory is walked by chunks (retention.cu) instead of row by row; 0: never (for tests and measurements).
+static int g_retention_chunk_rows = 128;
+extern "C" void kb_retention_chunk_rows(int rows) { g_retention_chunk_rows = rows >= 0 ? rows : 128; }
+static bool by_chunks(int longest) { return g_retention_chunk_rows > 0 && longest >= g_retention_chunk_rows; }
+
+// Floats of scratch kb_retention_scan takes for a step of `rows` rows whose longest portion has `longest`.
+extern "C" long long kb_retention_scratch_floats(int rows, int entries, int longest, int heads, int d, int e) {
+    return kb_decay_scan_scratch_floats(rows, heads, d, e, SCAN_FIXED) + (by_chunks(longest) ? retention_chunk_floats(rows, entries, heads, d, e) : 0);
+}
+
+// The read-out [rows, heads, e] of a matrix memory with a fixed decay a head behind rotated queries and keys. `longest`: the
+// most rows a request brings (every request's rows lie behind the earlier requests').
 extern "C" int kb_retention_scan(float* out, float* scratch, const void* src, int in_dt, int splits, long long split_stride, int row_width,
                                  int q_off, int k_off, int v_off, const float* decay, const float* cos_sin, int rotary, float k_scale,
                                  float* state, int n_slots, const int* entry_start, const int* entry_end, const int* slots, int entries,
-                                 int rows, int heads, int d, int e, void* stream) {
+                                 int rows, int longest, int heads, int d, int e, void* stream) {
     if (int err = scan_common_checks("retention", src, splits, split_stride, row_width, rows, entries, heads, d, e, state, n_slots, entry_start, entry_end, slots))
         return err;
     const long long nq = (long long)heads * d, nv = (long long)heads * e;
@@ -966,6 +983,9 @@ extern "C" int kb_retention_scan(float* out, float* scratch, const void* src, in
     else if (in_dt == KB_DT_BF16) retention_prep_kernel<bf16><<<rows, 256, 0, s>>>(Src<bf16>{(const bf16*)src, splits, (size_t)split_stride}, g, in);
     else return fail("retention: dtype code %d is not known", in_dt);
     if (int err = check_launch("retention prep")) return err;
+    if (by_chunks(longest))
+        return run_retention_chunks(out, in.vec, in.val, in.scal, decay, in.scal + (size_t)rows * heads * 2, state, n_slots, entry_start, entry_end,
+                                    slots, entries, longest, heads, d, e, s);
     return run_decay_scan(out, in, state, n_slots, entry_start, entry_end, slots, entries, heads, d, e, SCAN_FIXED, decay, s);
 }
 

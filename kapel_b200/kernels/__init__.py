@@ -62,7 +62,8 @@ def library():
                 lib.kb_last_error.restype = ctypes.c_char_p
                 for name in ("kb_gemm_bf16_scratch_floats", "kb_paged_attention_scratch_floats", "kb_attention_mma_scratch_floats", "kb_sample_scratch_floats",
                              "kb_mlstm_state_floats", "kb_delta_state_floats", "kb_delta_scratch_floats", "kb_pooled_attention_scratch_floats",
-                             "kb_pooled_attention_mma_scratch_floats", "kb_pooled_attention_mma_kept_floats", "kb_decay_scan_scratch_floats"):
+                             "kb_pooled_attention_mma_scratch_floats", "kb_pooled_attention_mma_kept_floats", "kb_decay_scan_scratch_floats",
+                             "kb_retention_scratch_floats"):
                     getattr(lib, name).restype = ctypes.c_longlong
                 lib.kb_launch_count.restype = ctypes.c_ulonglong
                 lib.kb_set_pdl(1 if PDL else 0)
@@ -1313,10 +1314,11 @@ def cdelta_scan(stacked, q_off: int, b_off: int, a1_off: int, a2: torch.Tensor, 
 
 
 def retention_scan(stacked, q_off: int, k_off: int, v_off: int, decay: torch.Tensor, cos_sin, rotary: int, k_scale: float,
-                   state: torch.Tensor, ranges, slots, entries: int, heads: int, d: int, e: int) -> torch.Tensor:
+                   state: torch.Tensor, ranges, slots, entries: int, longest: int, heads: int, d: int, e: int) -> torch.Tensor:
     """The read-out [rows, heads, e] (float32, not yet normed) of a matrix memory with a fixed decay a head
     (`decay` [heads]): S <- decay S + k v^T, o = S^T q, queries and keys turned by `cos_sin` [rows, rotary/2, 2]
-    (component i with i + rotary/2), keys then times `k_scale`; `state` [slots, heads e d]."""
+    (component i with i + rotary/2), keys then times `k_scale`; `state` [slots, heads e d]. `longest`: the most rows
+    a request brings; a long portion is walked by chunks of rows (`retention_chunk_rows`)."""
     src, dt, splits, stride, rows, width = _stacked(stacked, "retention input")
     _need(decay, "retention decays", torch.float32, (heads,))
     if rotary:
@@ -1326,12 +1328,18 @@ def retention_scan(stacked, q_off: int, k_off: int, v_off: int, decay: torch.Ten
         raise KernelError(f"retention: a state table of {tuple(state.shape)}, expected [slots, {heads * d * e}]")
     start, end = _ranges(ranges, slots, entries, "retention")
     out = _fresh((rows, heads, e), torch.float32, src.device)
-    scratch = _scan_scratch("fixed", rows, heads, d, e, src.device)
+    scratch = _fresh((max(1, int(library().kb_retention_scratch_floats(rows, int(entries), int(longest), heads, d, e))),), torch.float32, src.device)
     _check(library().kb_retention_scan(
         _ptr(out), _ptr(scratch), _ptr(src), dt, splits, ctypes.c_longlong(stride), width, int(q_off), int(k_off), int(v_off), _ptr(decay),
         _ptr(cos_sin if rotary else None), int(rotary), _f(k_scale), _ptr(state), int(state.shape[0]), _ptr(start), _ptr(end), _ptr(slots),
-        int(entries), rows, int(heads), int(d), int(e), _stream()))
+        int(entries), rows, int(longest), int(heads), int(d), int(e), _stream()))
     return out
+
+
+def retention_chunk_rows(n: int = -1) -> None:
+    """From how many rows of a request on `retention_scan` walks it by chunks: `n`, 0 for never, or -1 for the
+    launcher's own choice (for tests and measurements)."""
+    library().kb_retention_chunk_rows(int(n))
 
 
 def weighted_sum2(a, va: torch.Tensor, b=None, vb: Optional[torch.Tensor] = None, vc: Optional[torch.Tensor] = None) -> torch.Tensor:

@@ -63,8 +63,8 @@ class Retention(Part):
         nq, nv = s.num_heads * s.head_dim, self.inner_width
         rotary = self.position.rotary_dim
         o = K.retention_scan(stacked, base, base + nq, base + 2 * nq, self.decay, self.position.tables(batch) if rotary else None, rotary,
-                             s.head_dim ** -0.5, cache.state(), batch.entry_ranges(), batch.slots, batch.entries, s.num_heads, s.head_dim,
-                             s.v_head_dim)
+                             s.head_dim ** -0.5, cache.state(), batch.entry_ranges(), batch.slots, batch.entries, batch.longest_portion(), s.num_heads,
+                             s.head_dim, s.v_head_dim)
         return K.head_gate(o, stacked, base + 2 * nq + nv, None, True, s.eps, self.ctx.dtype, gate_act="silu", scale=scale, out=out, column=column,
                            pad_to=product_width(self.ctx, nv) if pad_to is None else pad_to)
 
