@@ -648,7 +648,8 @@ def design_point(which, z, steps, warmup, clocks, pk):
     K.enable_timing()
     per_kernel = {}
     for kind, fn in (("prefill", prefill_once), ("decode", decode_once)):
-        fn()
+        for _ in range(2):                 # the eager path's own memory, then a pass that finds it there
+            fn()
         K.timing_report()
         fn()
         rows = K.timing_report()
