@@ -58,7 +58,7 @@ CONFIGS = {
         lru_layer(24, 1, 1, None),
     ]}, 42),
     "C": ({"architecture": "Mukunex", "vocab": 64, "width": 32, "norm": {"eps": 1e-5}, "layers": [
-        parallel_layer(6, 2, 64, 64, 0.11, rotation(1000.0, 48, (2.0, 0.5, 8.0, 100)), 3, 40, 16, [0.5, 0.96875, 0.9990234375], rotation(300.0, 40), 1.0, 1.0, dense(40)),
+        parallel_layer(9, 3, 80, 80, 0.11, rotation(1000.0, 48, (2.0, 0.5, 8.0, 100)), 3, 40, 16, [0.5, 0.984375, 0.998046875], rotation(300.0, 40), 1.0, 1.0, dense(40)),
         lru_layer(16, 2, 7, None),
         delta_layer(3, 3, 8, 24, 4, 20, 1, dense(16)),
         parallel_layer(2, 1, 32, 32, 0.2, rotation(50.0, 2), 2, 16, 16, [0.75, 0.0], rotation(20.0, 4), -0.5, 1.5, None),
@@ -271,7 +271,7 @@ def attend(way, cache, q, rows, scale, sinks):
 
 
 @pytest.mark.parametrize("way", WAYS)
-@pytest.mark.parametrize("H,G,d", [(6, 2, 64), (4, 4, 128), (16, 1, 32), (3, 1, 48)])
+@pytest.mark.parametrize("H,G,d", [(9, 3, 80), (10, 2, 64), (4, 4, 128), (16, 1, 32), (3, 1, 48)])
 def test_attention_with_a_sink_on_every_kernel(way, H, G, d):
     rng = np.random.default_rng(H * d)
     dtype = torch.float32 if way == "rows f32" else torch.bfloat16
@@ -378,7 +378,7 @@ def test_convolution_with_biases_before_and_after(channels, taps):
 
 
 @pytest.mark.parametrize("w_dtype", [torch.float32, torch.bfloat16])
-@pytest.mark.parametrize("blocks,part", [(4, 24), (1, 7), (3, 80), (2, 128), (5, 130), (30, 1)])
+@pytest.mark.parametrize("blocks,part", [(4, 24), (1, 7), (3, 88), (2, 128), (5, 130), (30, 1)])
 def test_recurrent_units_gates_in_true_32_bit(blocks, part, w_dtype):
     """Few rows and many; the weights in both dtypes, the inputs never rounded."""
     from kapel_b200 import kernels as K
@@ -480,7 +480,7 @@ def test_retention_in_portions_and_token_by_token(H, d, e, rotary, scan_columns,
 
     rng = np.random.default_rng(d + e)
     nq, nv = H * d, H * e
-    decay = ([0.9990234375, 0.75, 1.0, 0.0])[:H] if H > 1 else [0.96875]
+    decay = ([0.998046875, 0.75, 1.0, 0.0])[:H] if H > 1 else [0.984375]
     rot = {"base": 70.0, "dims": rotary}
     data, want = {}, {}
     for name, T in LENGTHS.items():
