@@ -4,6 +4,7 @@ from .gemma2 import ConfigError, Gemma2Config
 from .kofutar import KofutarConfig
 from .lokedra import LokedraConfig
 from .mukunex import MukunexConfig
+from .sopalorn import SopalornConfig
 from .teluzen import TeluzenConfig
 from .registry import (
     architectures,
@@ -40,5 +41,6 @@ from .spec import (
     RopeBands,
     RopeScaling,
     ScheduleEntry,
+    StreamsSpec,
     default_schedule,
 )

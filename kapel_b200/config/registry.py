@@ -17,6 +17,7 @@ from .gemma2 import ConfigError, Gemma2Config
 from .kofutar import KofutarConfig
 from .lokedra import LokedraConfig
 from .mukunex import MukunexConfig
+from .sopalorn import SopalornConfig
 from .teluzen import TeluzenConfig
 
 _ARCHITECTURES: Dict[str, type] = {}
@@ -106,3 +107,4 @@ register_architecture(KofutarConfig, KofutarConfig.architecture, KofutarConfig.m
 register_architecture(TeluzenConfig, TeluzenConfig.architecture, TeluzenConfig.model_type)
 register_architecture(LokedraConfig, LokedraConfig.architecture, LokedraConfig.model_type)
 register_architecture(MukunexConfig, MukunexConfig.architecture, MukunexConfig.model_type)
+register_architecture(SopalornConfig, SopalornConfig.architecture, SopalornConfig.model_type)

@@ -17,13 +17,14 @@ from typing import Mapping, Optional, Tuple
 @dataclass(frozen=True)
 class NormSpec:
     """y = x / sqrt(mean(x^2) + eps) * (offset + w) for kind "rms"; kind "layer" takes the row's mean
-    off first: y = (x - mean) / sqrt(mean((x - mean)^2) + eps) * (offset + w), without a bias."""
+    off first: y = (x - mean) / sqrt(mean((x - mean)^2) + eps) * (offset + w), plus the tensor `bias` where one is named."""
 
     width: int
     eps: float
     offset: float
     weight: str                      # tensor name
     kind: str = "rms"
+    bias: Optional[str] = None
 
 
 @dataclass(frozen=True)
@@ -102,6 +103,8 @@ class AttentionSpec:
 
     `sink`: e^(sink[head]) joins the softmax's denominator (role sink [heads]; no key, no value, not scaled).
     `gate_by_head` (with `gated`): the gate is one number a head (g [heads, hidden]).
+    `borrows_kv`: the layer has no keys and values of its own (no roles k, v, no key norm); its runs are scheduled on another
+    layer's cache (`ScheduleEntry.cache_of`), whose kv heads, sizes and rotation are this layer's.
     """
 
     hidden: int
@@ -136,6 +139,7 @@ class AttentionSpec:
     out_bias: bool = False
     sink: bool = False
     gate_by_head: bool = False
+    borrows_kv: bool = False
 
 
 @dataclass(frozen=True)
@@ -223,9 +227,11 @@ class RetentionSpec:
     """Linear attention with a fixed decay a head (retention): a matrix memory S [head_dim, v_head_dim] a
     head and request.
 
-    q, k [heads, head_dim] turned by `position`, k then times head_dim^-1/2; v [heads, v_head_dim].
-    S <- `decay`[head] S + k v^T; o = S^T q, no softmax and no denominator. Each head's o is divided by its
-    root mean square (`eps`, no weight), times silu(g h), then o. `weights`: q, k, v, g, o.
+    q, k [heads, head_dim] and v [heads, v_head_dim] from the input through `activation` ("none" or "silu"), q and k turned
+    by `position`, k then times `key_scale` (None: head_dim^-1/2). S <- `decay`[head] S + k v^T; o = S^T q, no softmax and no
+    denominator. Each head's o is divided by its root mean square (`eps`, no weight), or with `whole_norm` the heads' o
+    together by theirs, times the weight `norm` [heads v_head_dim]; then times `gate`(g h) ("silu" or "sigmoid"), then o.
+    `weights`: q, k, v, g, o, and norm where used.
     """
 
     hidden: int
@@ -236,6 +242,10 @@ class RetentionSpec:
     eps: float
     position: PositionSpec
     weights: Mapping[str, str]
+    activation: str = "none"
+    key_scale: Optional[float] = None
+    whole_norm: bool = False
+    gate: str = "silu"
     kind: str = "retention"
 
 
@@ -305,12 +315,15 @@ class ForgetGateSpec:
 @dataclass(frozen=True)
 class ParallelMixerSpec:
     """Two mixers side by side that read the same input: `left_scale` left(h) + `right_scale` right(h).
-    Each keeps its own pages and state; at most one of them may ask for pages."""
+    Each keeps its own pages and state; at most one of them may ask for pages. With `left_norm` and `right_norm` (RMS norms over
+    the model's width, one eps) each side's result is normed before it is scaled and added."""
 
     left: object
     right: object
     left_scale: float
     right_scale: float
+    left_norm: Optional[NormSpec] = None
+    right_norm: Optional[NormSpec] = None
     kind: str = "parallel"
 
 
@@ -351,6 +364,8 @@ class MoESpec:
     weights by their sum. `weights`: router, correction (or absent), and the patterns `up` and
     `down` with `{e}` for the expert's number. The gated activation "clamped_swish" with `limit` L and
     `swish_alpha` a: g = min(gate h, L), u = clamp(up h, -L, L), the unit is g sigmoid(a g) (u + 1).
+    The router has `identity` outputs more than there are experts: the last ones are experts that give back their input.
+    The weights are multiplied by `route_scale` at the end.
     """
 
     hidden: int
@@ -368,17 +383,22 @@ class MoESpec:
     shared: Optional[object] = None
     limit: Optional[float] = None
     swish_alpha: float = 1.702
+    identity: int = 0
+    route_scale: float = 1.0
     kind: str = "moe"
 
 
 @dataclass(frozen=True)
 class GatedMLPSpec:
-    """down(act(gate(h)) * up(h)); `activation` is "gelu_tanh" or "silu"."""
+    """down(act(gate(h)) * up(h)); `activation` is "gelu_tanh" or "silu", or "clamped_swish" with `limit` and `swish_alpha`
+    (the bounded unit of `MoESpec`)."""
 
     hidden: int
     intermediate: int
     activation: str
     weights: Mapping[str, str]       # roles gate, up, down
+    limit: Optional[float] = None
+    swish_alpha: float = 1.702
     kind: str = "gated_mlp"
 
 
@@ -394,6 +414,18 @@ class MLPSpec:
 
 
 @dataclass(frozen=True)
+class StreamsSpec:
+    """How a sublayer reads and writes `count` residual streams x_s: u = sum_s in[s] x_s; y = sublayer(norm(u)); then, all at
+    once from the old ones, x_t <- sum_s mix[s, t] x_s + out[t] y. Tensor names: `read` [count], `write` [count],
+    `mix` [count, count]."""
+
+    count: int
+    read: str
+    write: str
+    mix: str
+
+
+@dataclass(frozen=True)
 class BlockSpec:
     """The arrangement of one layer.
 
@@ -406,6 +438,8 @@ class BlockSpec:
     multiplied, channel by channel, by a weight [hidden] (the second is absent without a feed-forward);
     with `shift` (a tensor [hidden]) the mixer, and only the mixer, reads h_t + (h_(t-1) - h_t) * shift,
     h_(t-1) the row before (zeros for a request's first row), which is state of a request.
+    kind "streams" (hyper-connections): instead of one residual there are several, and `streams` says for each sublayer (the
+    second None without a feed-forward) how it reads and writes them; norms `pre_mixer` and `pre_ffn`; `scales` as above.
     """
 
     mixer: object
@@ -414,6 +448,7 @@ class BlockSpec:
     kind: str = "sandwich"
     scales: Optional[Tuple[str, Optional[str]]] = None
     shift: Optional[str] = None
+    streams: Optional[Tuple[StreamsSpec, Optional[StreamsSpec]]] = None
 
 
 @dataclass(frozen=True)
@@ -466,13 +501,19 @@ class EmbedSpec:
 
 @dataclass(frozen=True)
 class HeadSpec:
+    """Logits: `scale` times the product of the final norm's output and the table, then the soft cap where one is given."""
+
     weight: str                      # the table [vocab, hidden]; the embedding's when tied
     softcap: Optional[float]
     kind: str = "vocab_head"
+    scale: float = 1.0
 
 
 @dataclass(frozen=True)
 class ModelSpec:
+    """`streams` > 0: every layer's block is of kind "streams"; that many copies of the embedding's output start, and their sum
+    goes to the final norm."""
+
     architecture: str
     vocab_size: int
     hidden_size: int
@@ -482,6 +523,7 @@ class ModelSpec:
     final_norm: NormSpec
     head: HeadSpec
     max_positions: Optional[int] = None
+    streams: int = 0
     extra: Mapping[str, object] = field(default_factory=dict)
 
 

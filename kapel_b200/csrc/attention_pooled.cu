@@ -511,7 +511,8 @@ extern "C" int kb_proj_rope_append(const void* src, int src_dt, int splits, long
                                    int neighbours, const float* v_other, const void* lambda, float* v_keep, const int* lines,
                                    void* q_out, void* k_table, void* v_table, int out_dt, int rows, int hq, int hkv, int d, int dv,
                                    int write_kv, long long table_lines, int page_size, void* stream) {
-    KB_REQUIRE(rows >= 0 && hq > 0 && hkv > 0 && d > 0 && dv > 0, "proj_rope_append: rows %d, heads %d / %d, sizes %d / %d", rows, hq, hkv, d, dv);
+    KB_REQUIRE(rows >= 0 && hq > 0 && hkv >= 0 && d > 0 && dv > 0, "proj_rope_append: rows %d, heads %d / %d, sizes %d / %d", rows, hq, hkv, d, dv);
+    KB_REQUIRE(hkv > 0 || (!write_kv && v_keep == nullptr && v_other == nullptr), "proj_rope_append: a projection of queries alone has no keys or values to keep");
     KB_REQUIRE(splits >= 1 && row_width > 0, "proj_rope_append: %d slices of rows of %d", splits, row_width);
     KB_REQUIRE(q_off >= 0 && k_off >= 0 && v_off >= 0 && q_off + hq * d <= row_width && k_off + hkv * d <= row_width && v_off + hkv * dv <= row_width,
                "proj_rope_append: offsets %d, %d, %d do not fit rows of %d", q_off, k_off, v_off, row_width);

@@ -14,15 +14,15 @@ KB_TIMELINE_ARRAY(elementwise) // slots: kind 3 rotation and append (rows, slice
 // ---------------------------------------------------------------------------------------
 // x[r, :] = table[ids[r], :] * scale, in 32-bit. An id outside the table gives a row of NaN.
 // With a table of learned positions, its row positions[r] is added (not scaled); a position outside
-// that table (a row of no token) adds nothing.
+// that table (a row of no token) adds nothing. The row is written `copies` times, side by side.
 template <typename T>
 __global__ void embed_kernel(float* __restrict__ out, const T* __restrict__ table, const int* __restrict__ ids,
                              int rows, int width, int vocab, float scale, const T* __restrict__ pos_table,
-                             const int* __restrict__ positions, int max_positions) {
-    const int r = blockIdx.x;
+                             const int* __restrict__ positions, int max_positions, int copies) {
+    const int r = blockIdx.x / copies;
     if (r >= rows) return;
     const int id = ids[r];
-    float* o = out + (size_t)r * width;
+    float* o = out + (size_t)blockIdx.x * width;
     if (id < 0 || id >= vocab) {
         for (int i = threadIdx.x; i < width; i += blockDim.x) o[i] = __int_as_float(0x7fc00000);
         return;
@@ -382,16 +382,17 @@ extern "C" int kb_poison(void* x, int dt, long long n, void* stream) {
 }
 
 extern "C" int kb_embed(float* out, const void* table, int table_dt, const int* ids, int rows, int width,
-                        int vocab, float scale, const void* pos_table, const int* positions, int max_positions, void* stream) {
+                        int vocab, float scale, const void* pos_table, const int* positions, int max_positions, int copies, void* stream) {
+    KB_REQUIRE(copies >= 1 && (long long)rows * copies <= 0x7fffffffll, "embed: %d rows %d times", rows, copies);
     KB_REQUIRE(rows >= 0 && width > 0 && vocab > 0, "embed: rows %d, width %d, vocab %d", rows, width, vocab);
     KB_REQUIRE(pos_table == nullptr || (positions != nullptr && max_positions > 0), "embed: a table of positions without the rows' positions");
     if (rows == 0) return 0;
     cudaStream_t s = (cudaStream_t)stream;
     const int threads = width >= 1024 ? 256 : 128;
     if (table_dt == KB_DT_F32)
-        embed_kernel<float><<<rows, threads, 0, s>>>(out, (const float*)table, ids, rows, width, vocab, scale, (const float*)pos_table, positions, max_positions);
+        embed_kernel<float><<<rows * copies, threads, 0, s>>>(out, (const float*)table, ids, rows, width, vocab, scale, (const float*)pos_table, positions, max_positions, copies);
     else if (table_dt == KB_DT_BF16)
-        embed_kernel<bf16><<<rows, threads, 0, s>>>(out, (const bf16*)table, ids, rows, width, vocab, scale, (const bf16*)pos_table, positions, max_positions);
+        embed_kernel<bf16><<<rows * copies, threads, 0, s>>>(out, (const bf16*)table, ids, rows, width, vocab, scale, (const bf16*)pos_table, positions, max_positions, copies);
     else
         return fail("embed: table dtype code %d is not known", table_dt);
     return check_launch("embed");

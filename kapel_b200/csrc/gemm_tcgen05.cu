@@ -131,8 +131,15 @@ __device__ __forceinline__ void tc_ld16(uint32_t taddr, uint32_t (&r)[16]) {
 }
 
 // Epilogues, chosen at compile time so that each kernel carries only its own code:
-// 0 none, 1 soft cap c * tanh(x / c), 2 and 3 the gated unit gelu_tanh(gate) * up and silu(gate) * up.
-constexpr int EPI_NONE = 0, EPI_SOFTCAP = 1, EPI_GLU_GELU = 2, EPI_GLU_SILU = 3;
+// 0 none, 1 soft cap c * tanh(x / c), 2 and 3 the gated unit gelu_tanh(gate) * up and silu(gate) * up, 4 the unit with
+// both halves bounded, g sigmoid(alpha g) (u + 1) with g = min(gate, cap) and u = clamp(up, -cap, cap).
+constexpr int EPI_NONE = 0, EPI_SOFTCAP = 1, EPI_GLU_GELU = 2, EPI_GLU_SILU = 3, EPI_GLU_BOUNDED = 4;
+__host__ __device__ constexpr bool epi_glu(int epi) { return epi == EPI_GLU_GELU || epi == EPI_GLU_SILU || epi == EPI_GLU_BOUNDED; }
+__device__ __forceinline__ float glu_bounded(float g, float u, float cap, float alpha) {
+    g = fminf(g, cap);
+    u = fminf(fmaxf(u, -cap), cap);
+    return g / (1.f + __expf(-alpha * g)) * (u + 1.f);
+}
 
 __device__ __forceinline__ uint4 tc_pack8(const float (&v)[8]) {
     uint4 o;
@@ -173,9 +180,9 @@ __device__ __forceinline__ void tc_store8(void* __restrict__ c, int c_dt, size_t
 // accumulator's columns 0-127 are gates and 128-255 the matching ups, C is [m, n] with n the unit's
 // width, and n0 counts in outputs.
 template <int EPI>
-__device__ __forceinline__ void tc_epilogue(uint32_t lanes, int row, int n0, void* __restrict__ c, int c_dt, int m, int n, float cap) {
+__device__ __forceinline__ void tc_epilogue(uint32_t lanes, int row, int n0, void* __restrict__ c, int c_dt, int m, int n, float cap, float alpha = 0.f) {
     const bool vec = (c_dt == KB_DT_BF16) ? (n % 8 == 0) : (n % 4 == 0);
-    if constexpr (EPI == EPI_GLU_GELU || EPI == EPI_GLU_SILU) {
+    if constexpr (epi_glu(EPI)) {
         for (int c0 = 0; c0 < 128; c0 += 16) {
             if (n0 + c0 >= n) break;                            // the same for the whole warp
             uint32_t g[16], u[16];
@@ -189,8 +196,8 @@ __device__ __forceinline__ void tc_epilogue(uint32_t lanes, int row, int n0, voi
                 float v[8];
 #pragma unroll
                 for (int j = 0; j < 8; ++j) {
-                    const float x = __uint_as_float(g[h + j]);
-                    v[j] = (EPI == EPI_GLU_GELU ? gelu_tanh(x) : silu(x)) * __uint_as_float(u[h + j]);
+                    const float x = __uint_as_float(g[h + j]), up = __uint_as_float(u[h + j]);
+                    v[j] = EPI == EPI_GLU_BOUNDED ? glu_bounded(x, up, cap, alpha) : (EPI == EPI_GLU_GELU ? gelu_tanh(x) : silu(x)) * up;
                 }
                 const int col = n0 + c0 + h;
                 tc_store8(c, c_dt, (size_t)row * n + col, col, n, vec && col + 8 <= n, v);
@@ -358,7 +365,7 @@ __device__ __forceinline__ void tp_arrive_on_first(uint64_t* bar) {
 template <int EPI>
 __global__ void __cluster_dims__(2, 1, 1) __launch_bounds__(TC_THREADS, 1)
 gemm_tcgen05_pair_persistent_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant__ CUtensorMap map_w,
-                                    void* __restrict__ c, int c_dt, int m, int n, int k, float cap) {
+                                    void* __restrict__ c, int c_dt, int m, int n, int k, float cap, float alpha) {
     extern __shared__ unsigned char tc_smem_raw[];
     unsigned char* smem = reinterpret_cast<unsigned char*>(((uintptr_t)tc_smem_raw + 1023) & ~(uintptr_t)1023);
     uint64_t* full = reinterpret_cast<uint64_t*>(smem + TPP_STAGES * TP_STAGE_BYTES);
@@ -450,7 +457,7 @@ gemm_tcgen05_pair_persistent_kernel(const __grid_constant__ CUtensorMap map_a, c
             const int n0 = (t / m_pairs) * tile_cols;
             if (!__all_sync(0xffffffffu, tc_mbar_wait(acc_full + acc, (uint32_t)(i >> 1) & 1u))) { failed = true; break; }
             tc_fence_after();
-            tc_epilogue<EPI>(tmem + ((uint32_t)(quarter * 32) << 16) + (uint32_t)(acc * 256), m0 + quarter * 32 + lane, n0, c, c_dt, m, n, cap);
+            tc_epilogue<EPI>(tmem + ((uint32_t)(quarter * 32) << 16) + (uint32_t)(acc * 256), m0 + quarter * 32 + lane, n0, c, c_dt, m, n, cap, alpha);
             tc_fence_before();
             __syncwarp();
             if (lane == 0) tp_arrive_on_first(acc_empty + acc);
@@ -649,7 +656,7 @@ template <int NP> struct SkGlu {
 template <int NP>
 __global__ void __launch_bounds__(TC_THREADS, 1)
 gemm_skinny_glu_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant__ CUtensorMap map_x,
-                       bf16* __restrict__ c, int m, int n, int k, int act KB_TL_PARAM) {
+                       bf16* __restrict__ c, int m, int n, int k, int act, float cap, float alpha KB_TL_PARAM) {
     using G = SkGlu<NP>;
     constexpr int STAGES = G::STAGES, STAGE = G::STAGE;
     constexpr uint32_t IDESC = (1u << 4) | (1u << 7) | (1u << 10) | ((uint32_t)(NP >> 3) << 17) | ((uint32_t)(SK2_BM >> 4) << 24);
@@ -774,7 +781,7 @@ gemm_skinny_glu_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_c
                     const int j = j0 + 2 * u;               // the even row; the up warps take the odd one after it
                     const float g = gates ? v[j] : xch[(j + 1) * SKG_ROWS + f];
                     const float up = gates ? xch[j * SKG_ROWS + f] : v[j + 1];
-                    o[u] = (act == 0 ? gelu_tanh(g) : silu(g)) * up;
+                    o[u] = act == 2 ? glu_bounded(g, up, cap, alpha) : (act == 0 ? gelu_tanh(g) : silu(g)) * up;
                 }
 #pragma unroll
                 for (int u = 0; u < 4; ++u) {
@@ -795,14 +802,14 @@ gemm_skinny_glu_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_c
 }
 
 template <int NP>
-static int launch_skinny_glu(const CUtensorMap& map_w, const CUtensorMap& map_x, bf16* c, int m, int n, int k, int act, cudaStream_t s) {
+static int launch_skinny_glu(const CUtensorMap& map_w, const CUtensorMap& map_x, bf16* c, int m, int n, int k, int act, float cap, float alpha, cudaStream_t s) {
     static bool attr_set = false;
     if (!attr_set) {
         const cudaError_t e = cudaFuncSetAttribute(gemm_skinny_glu_kernel<NP>, cudaFuncAttributeMaxDynamicSharedMemorySize, SkGlu<NP>::SMEM);
         if (e != cudaSuccess) return fail("gemm_skinny_glu: cannot have %d bytes of shared memory: %s", SkGlu<NP>::SMEM, cudaGetErrorString(e));
         attr_set = true;
     }
-    launch_dependent_if(m <= DEPENDENT_ROWS, gemm_skinny_glu_kernel<NP>, dim3((n + SKG_ROWS - 1) / SKG_ROWS), dim3(TC_THREADS), (size_t)SkGlu<NP>::SMEM, s, map_w, map_x, c, m, n, k, act KB_TL_SLOT(gemm, 1, n, k));
+    launch_dependent_if(m <= DEPENDENT_ROWS, gemm_skinny_glu_kernel<NP>, dim3((n + SKG_ROWS - 1) / SKG_ROWS), dim3(TC_THREADS), (size_t)SkGlu<NP>::SMEM, s, map_w, map_x, c, m, n, k, act, cap, alpha KB_TL_SLOT(gemm, 1, n, k));
     return check_launch("gemm_skinny_glu");
 }
 
@@ -866,18 +873,18 @@ static int launch_single(const CUtensorMap& map_a, const CUtensorMap& map_w, voi
 // n counts output columns (the gated unit's width with a gated epilogue).
 template <int EPI>
 static int launch_pair(const CUtensorMap& map_a, const CUtensorMap& map_w, void* c, int c_dt, int m, int n, int k, float cap,
-                       cudaStream_t s) {
+                       cudaStream_t s, float alpha = 0.f) {
     static bool attr_set = false;
     if (!attr_set) {
         const cudaError_t e = cudaFuncSetAttribute(gemm_tcgen05_pair_persistent_kernel<EPI>, cudaFuncAttributeMaxDynamicSharedMemorySize, tp_smem_bytes(TPP_STAGES));
         if (e != cudaSuccess) return fail("gemm_tcgen05_pair: cannot have %d bytes of shared memory: %s", tp_smem_bytes(TPP_STAGES), cudaGetErrorString(e));
         attr_set = true;
     }
-    constexpr int tile_cols = (EPI == EPI_GLU_GELU || EPI == EPI_GLU_SILU) ? TP_BN_HALF : 2 * TP_BN_HALF;
+    constexpr int tile_cols = epi_glu(EPI) ? TP_BN_HALF : 2 * TP_BN_HALF;
     const long long tiles = (long long)((m + 2 * TC_BM - 1) / (2 * TC_BM)) * ((n + tile_cols - 1) / tile_cols);
     const int pairs = skinny_sms() / 2;
     const int clusters = tiles < pairs ? (int)tiles : pairs;
-    launch_dependent_if(false, gemm_tcgen05_pair_persistent_kernel<EPI>, dim3(2 * clusters), dim3(TC_THREADS), (size_t)tp_smem_bytes(TPP_STAGES), s, map_a, map_w, c, c_dt, m, n, k, cap);
+    launch_dependent_if(false, gemm_tcgen05_pair_persistent_kernel<EPI>, dim3(2 * clusters), dim3(TC_THREADS), (size_t)tp_smem_bytes(TPP_STAGES), s, map_a, map_w, c, c_dt, m, n, k, cap, alpha);
     return check_launch("gemm_tcgen05_pair");
 }
 
@@ -977,36 +984,37 @@ extern "C" int kb_gemm_tcgen05_split(float* partial, const void* a, const void* 
 }
 
 // The gated unit in the product's epilogue: a bf16 [m,k]; w bf16 [2 n, k], gate rows then up rows;
-// c = act(a . gate^T) * (a . up^T), bf16 [m, n]; act 0 gelu_tanh, 1 silu. The gate and the up sums
-// meet in 32-bit, before any rounding to bfloat16.
-extern "C" int kb_gemm_tcgen05_glu(void* c, const void* a, const void* w, int m, int n, int k, int act, void* stream) {
+// c = act(a . gate^T) * (a . up^T), bf16 [m, n]; act 0 gelu_tanh, 1 silu, 2 the bounded unit of `cap` and `alpha`. The gate
+// and the up sums meet in 32-bit, before any rounding to bfloat16.
+extern "C" int kb_gemm_tcgen05_glu(void* c, const void* a, const void* w, int m, int n, int k, int act, float cap, float alpha, void* stream) {
     KB_REQUIRE(m > 0 && n > 0 && k > 0, "gemm_tcgen05_glu: m %d, n %d, k %d", m, n, k);
     KB_REQUIRE(k % 8 == 0, "gemm_tcgen05_glu: k = %d must be a multiple of 8 (16-byte rows)", k);
-    KB_REQUIRE(act == 0 || act == 1, "gemm_tcgen05_glu: activation code %d is not known (0 gelu_tanh, 1 silu)", act);
+    KB_REQUIRE(act == 0 || act == 1 || (act == 2 && cap > 0.f), "gemm_tcgen05_glu: activation code %d is not known (0 gelu_tanh, 1 silu, 2 bounded by %g)", act, cap);
     KB_REQUIRE(((uintptr_t)a & 15) == 0 && ((uintptr_t)w & 15) == 0 && ((uintptr_t)c & 15) == 0, "gemm_tcgen05_glu: operands must be 16-byte aligned");
     CUtensorMap map_a, map_w;
     if (int e = encode_map_bf16(&map_a, a, m, k, k, TC_BM)) return e;
     if (int e = encode_map_bf16(&map_w, w, 2ull * n, k, k, TP_BN_HALF)) return e;
     cudaStream_t s = (cudaStream_t)stream;
+    if (act == 2) return launch_pair<EPI_GLU_BOUNDED>(map_a, map_w, c, KB_DT_BF16, m, n, k, cap, s, alpha);
     return act == 0 ? launch_pair<EPI_GLU_GELU>(map_a, map_w, c, KB_DT_BF16, m, n, k, 0.f, s)
                     : launch_pair<EPI_GLU_SILU>(map_a, map_w, c, KB_DT_BF16, m, n, k, 0.f, s);
 }
 
 // The gated unit for up to 64 rows: a bf16 [m,k]; w bf16 [2 n, k], gate rows then up rows;
-// c = act(a . gate^T) * (a . up^T), bf16 [m, n]; act 0 gelu_tanh, 1 silu.
-extern "C" int kb_gemm_skinny_glu(void* c, const void* a, const void* w, int m, int n, int k, int act, void* stream) {
+// c = act(a . gate^T) * (a . up^T), bf16 [m, n]; act 0 gelu_tanh, 1 silu, 2 the bounded unit of `cap` and `alpha`.
+extern "C" int kb_gemm_skinny_glu(void* c, const void* a, const void* w, int m, int n, int k, int act, float cap, float alpha, void* stream) {
     KB_REQUIRE(m > 0 && m <= 64 && n > 0 && k > 0, "gemm_skinny_glu: m %d (1..64), n %d, k %d", m, n, k);
     KB_REQUIRE(k % 8 == 0, "gemm_skinny_glu: k = %d must be a multiple of 8 (16-byte rows)", k);
-    KB_REQUIRE(act == 0 || act == 1, "gemm_skinny_glu: activation code %d is not known (0 gelu_tanh, 1 silu)", act);
+    KB_REQUIRE(act == 0 || act == 1 || (act == 2 && cap > 0.f), "gemm_skinny_glu: activation code %d is not known (0 gelu_tanh, 1 silu, 2 bounded by %g)", act, cap);
     KB_REQUIRE(((uintptr_t)a & 15) == 0 && ((uintptr_t)w & 15) == 0, "gemm_skinny_glu: operands must be 16-byte aligned");
     const int np = m <= 16 ? 16 : (m <= 32 ? 32 : 64);
     CUtensorMap map_w, map_x;
     if (int e = encode_map_bf16(&map_w, w, 2ull * n, k, k, SKG_ROWS)) return e;
     if (int e = encode_map_bf16(&map_x, a, m, k, k, np)) return e;
     cudaStream_t s = (cudaStream_t)stream;
-    if (np == 16) return launch_skinny_glu<16>(map_w, map_x, (bf16*)c, m, n, k, act, s);
-    if (np == 32) return launch_skinny_glu<32>(map_w, map_x, (bf16*)c, m, n, k, act, s);
-    return launch_skinny_glu<64>(map_w, map_x, (bf16*)c, m, n, k, act, s);
+    if (np == 16) return launch_skinny_glu<16>(map_w, map_x, (bf16*)c, m, n, k, act, cap, alpha, s);
+    if (np == 32) return launch_skinny_glu<32>(map_w, map_x, (bf16*)c, m, n, k, act, cap, alpha, s);
+    return launch_skinny_glu<64>(map_w, map_x, (bf16*)c, m, n, k, act, cap, alpha, s);
 }
 
 // Partial sums the skinny kernel leaves for a weight [n, k] and up to 64 rows (1: it writes the result itself).

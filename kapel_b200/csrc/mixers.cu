@@ -118,6 +118,44 @@ __global__ void head_gate_kernel(TO* __restrict__ out, const TY* __restrict__ y,
         for (int c = heads * e + lane; c < fill_to; c += 32) Elem<TO>::store(out + (size_t)r * out_stride + c, 0.f);
 }
 
+// The same for wide heads (a whole row normed as one, say): one block a (row, head).
+template <typename TY, typename TS, typename TW, typename TO>
+__global__ void __launch_bounds__(1024)
+head_gate_wide_kernel(TO* __restrict__ out, const TY* __restrict__ y, const Src<TS> gate, int row_width, int g_off, const TW* __restrict__ w,
+                      int unit, float eps, int heads, int e, int out_stride, int fill_to, int act, int by_head, float scale) {
+    __shared__ float scratch[32];
+    const long long pair = blockIdx.x;
+    const long long r = pair / heads;
+    const int h = (int)(pair - r * heads);
+    const TY* yp = y + (size_t)pair * e;
+    float inv = 1.f;
+    if (unit) {
+        float ss = 0.f;
+        for (int c = threadIdx.x; c < e; c += blockDim.x) {
+            const float v = Elem<TY>::load(yp + c);
+            ss = fmaf(v, v, ss);
+        }
+        ss = block_sum(ss, scratch);
+        inv = 1.f / sqrtf(ss / (float)e + eps);
+    }
+    inv *= scale;
+    if (by_head && act != 2) {
+        const float z = gate.at((size_t)r * row_width + g_off + h);
+        inv *= act == 1 ? z / (1.f + expf(-z)) : 1.f / (1.f + expf(-z));
+    }
+    for (int c = threadIdx.x; c < e; c += blockDim.x) {
+        float v = Elem<TY>::load(yp + c) * inv;
+        if (w != nullptr) v *= Elem<TW>::load(w + (size_t)h * e + c);
+        if (act != 2 && !by_head) {
+            const float z = gate.at((size_t)r * row_width + g_off + (size_t)h * e + c);
+            v *= act == 1 ? z / (1.f + expf(-z)) : 1.f / (1.f + expf(-z));
+        }
+        Elem<TO>::store(out + (size_t)r * out_stride + (size_t)h * e + c, v);
+    }
+    if (h == heads - 1)
+        for (int c = heads * e + threadIdx.x; c < fill_to; c += blockDim.x) Elem<TO>::store(out + (size_t)r * out_stride + c, 0.f);
+}
+
 // One block a row; a warp takes head vectors in turn (queries, then keys, then values) through a
 // piece of shared memory of its own.
 template <typename TS, typename TW, typename TO>
@@ -532,8 +570,14 @@ extern "C" int kb_head_gate(void* out, int out_dt, const void* y, int y_dt, cons
     const long long pairs = rows * heads;
     const int warps = 4;
     const long long blocks = (pairs + warps - 1) / warps;
-    KB_REQUIRE(blocks <= 0x7fffffffll, "head_gate: too many rows for one launch");
+    KB_REQUIRE(pairs <= 0x7fffffffll, "head_gate: too many rows for one launch");
+    const int wide = e >= 512 ? (rows <= DEPENDENT_ROWS ? (e >= 1024 ? 1024 : 512) : 256) : 0;      // threads of a block a head; 0: a warp a head
 #define KB_HG(TY, TS, TW, TO)                                                                                       \
+    if (wide)                                                                                                       \
+        head_gate_wide_kernel<TY, TS, TW, TO><<<(unsigned)pairs, wide, 0, s>>>((TO*)out, (const TY*)y,                   \
+                                                                             Src<TS>{(const TS*)gate, splits, (size_t)split_stride}, \
+                                                                             row_width, g_off, (const TW*)w, unit, eps, heads, e, out_stride, fill_to, act, by_head, scale); \
+    else                                                                                                            \
     head_gate_kernel<TY, TS, TW, TO><<<(unsigned)blocks, warps * 32, 0, s>>>((TO*)out, (const TY*)y,                    \
                                                                              Src<TS>{(const TS*)gate, splits, (size_t)split_stride}, \
                                                                              row_width, g_off, (const TW*)w, unit, eps, pairs, heads, e, out_stride, fill_to, act, by_head, scale)

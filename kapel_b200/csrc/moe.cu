@@ -6,12 +6,14 @@
 //            s + correction; experts in equal groups of neighbours, a group's score the sum of its
 //            `group_top` largest choice scores, only the best `keep_groups` groups stay eligible;
 //            the `top` largest eligible choice scores are chosen (the lower number wins a tie) and
-//            weighted by s, optionally divided by their sum.
-//  sort      (token, k) pairs listed by expert, and the row tiles of the grouped products.
+//            weighted by s, optionally divided by their sum (+ 1e-20), times a number. Outputs of the router beyond the
+//            experts that have weights are identity experts.
+//  sort      (token, k) pairs listed by expert (identity experts left out), and the row tiles of the grouped products.
 //  product   out[pair] = act(A[row of pair] . W[expert of pair]^T): a block a (row tile of one
 //            expert, column tile); bfloat16 by mma.sync with 32-bit sums, float32 by FMA in
 //            ascending k. What a pair's row computes does not depend on its place in a tile.
-//  combine   out[token] = sum over k, in order, of weight[token, k] * y[token * top + k].
+//  combine   out[token] = sum over k, in order, of weight[token, k] * y[token * top + k]; an identity expert's y is the
+//            token's own input.
 #include "common.cuh"
 
 namespace kb {
@@ -25,7 +27,7 @@ template <typename TH>
 __global__ void __launch_bounds__(ROUTE_THREADS)
 moe_route_kernel(const TH* __restrict__ h, const float* __restrict__ router, const float* __restrict__ correction,
                  int* __restrict__ experts_out, float* __restrict__ weights_out, int width, int n_experts, int top, int groups,
-                 int keep_groups, int group_top, int softmax, int renormalize) {
+                 int keep_groups, int group_top, int softmax, int renormalize, float scale) {
     extern __shared__ float sm[];
     float* score = sm;                         // [E] s
     float* choice = sm + n_experts;            // [E] s + correction
@@ -127,11 +129,14 @@ moe_route_kernel(const TH* __restrict__ h, const float* __restrict__ router, con
         const float mx = w[0];
         float sum = 0.f;
         for (int t = 0; t < top; ++t) { w[t] = expf(w[t] - mx); sum += w[t]; }
-        for (int t = 0; t < top; ++t) w[t] /= sum;
+        for (int t = 0; t < top; ++t) w[t] = w[t] / sum * scale;
         return;
     }
-    if (renormalize && total > 0.f)
-        for (int t = 0; t < top; ++t) weights_out[(size_t)r * top + t] /= total;
+    if (renormalize || scale != 1.f)
+        for (int t = 0; t < top; ++t) {
+            float& w = weights_out[(size_t)r * top + t];
+            w = (renormalize ? w / (total + 1e-20f) : w) * scale;
+        }
 }
 
 // ------------------------------------------------------------------------------------------- sort
@@ -387,13 +392,19 @@ moe_grouped_bf16_kernel(const GroupedParams p) {
 // expert that every token uses.
 template <typename TO, typename TA>
 __global__ void moe_combine_kernel(TO* __restrict__ out, const float* __restrict__ y, const float* __restrict__ weights,
-                                   long long rows, int width, int top, const Src<TA> also) {
+                                   long long rows, int width, int top, const Src<TA> also, const int* __restrict__ experts, int real,
+                                   const void* __restrict__ self, int self_dt) {
     const long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
     if (i >= rows * width) return;
     const long long r = i / width;
     const int c = (int)(i - r * width);
     float acc = 0.f;
-    for (int t = 0; t < top; ++t) acc = fmaf(weights[r * top + t], y[((size_t)r * top + t) * width + c], acc);
+    if (experts != nullptr) {                                // experts from `real` on are the identity: their pairs have no row in y
+        const float own = self_dt == KB_DT_F32 ? static_cast<const float*>(self)[i] : Elem<bf16>::load(static_cast<const bf16*>(self) + i);
+        for (int t = 0; t < top; ++t) acc = fmaf(weights[r * top + t], experts[r * top + t] < real ? y[((size_t)r * top + t) * width + c] : own, acc);
+    } else {
+        for (int t = 0; t < top; ++t) acc = fmaf(weights[r * top + t], y[((size_t)r * top + t) * width + c], acc);
+    }
     if (also.p != nullptr) acc += also.at((size_t)i);
     Elem<TO>::store(out + i, acc);
 }
@@ -409,7 +420,7 @@ extern "C" int kb_moe_tile_rows(int dt, long long rows_an_expert) {
 
 extern "C" int kb_moe_route(int* experts, float* weights, const void* h, int h_dt, const float* router, const float* correction,
                             int rows, int width, int n_experts, int top, int groups, int keep_groups, int group_top,
-                            int softmax, int renormalize, void* stream) {
+                            int softmax, int renormalize, float scale, void* stream) {
     KB_REQUIRE(softmax >= 0 && softmax <= 2, "moe_route: scoring code %d is not known (0 sigmoid, 1 softmax, 2 softmax over the chosen)", softmax);
     KB_REQUIRE(rows >= 0 && width > 0 && n_experts > 0 && top > 0 && top <= n_experts, "moe_route: rows %d, width %d, %d experts, top %d", rows, width, n_experts, top);
     KB_REQUIRE(groups >= 1 && n_experts % groups == 0 && keep_groups >= 1 && keep_groups <= groups,
@@ -422,10 +433,10 @@ extern "C" int kb_moe_route(int* experts, float* weights, const void* h, int h_d
     cudaStream_t s = (cudaStream_t)stream;
     if (h_dt == KB_DT_F32)
         moe_route_kernel<float><<<rows, ROUTE_THREADS, smem, s>>>((const float*)h, router, correction, experts, weights, width, n_experts, top,
-                                                                  groups, keep_groups, group_top, softmax, renormalize);
+                                                                  groups, keep_groups, group_top, softmax, renormalize, scale);
     else if (h_dt == KB_DT_BF16)
         moe_route_kernel<bf16><<<rows, ROUTE_THREADS, smem, s>>>((const bf16*)h, router, correction, experts, weights, width, n_experts, top,
-                                                                 groups, keep_groups, group_top, softmax, renormalize);
+                                                                 groups, keep_groups, group_top, softmax, renormalize, scale);
     else return fail("moe_route: dtype code %d is not known", h_dt);
     return check_launch("moe_route");
 }
@@ -489,7 +500,10 @@ extern "C" int kb_moe_grouped(void* out, int out_dt, const void* a, const void* 
 }
 
 extern "C" int kb_moe_combine(void* out, int out_dt, const float* y, const float* weights, long long rows, int width, int top,
-                              const void* also, int also_dt, int also_splits, long long also_stride, void* stream) {
+                              const void* also, int also_dt, int also_splits, long long also_stride, const int* experts, int real,
+                              const void* self, int self_dt, void* stream) {
+    KB_REQUIRE(experts == nullptr || (self != nullptr && real >= 0 && (self_dt == KB_DT_F32 || self_dt == KB_DT_BF16)),
+               "moe_combine: identity experts without the rows they give back");
     KB_REQUIRE(rows >= 0 && width > 0 && top > 0, "moe_combine: rows %lld, width %d, top %d", rows, width, top);
     KB_REQUIRE(also == nullptr || also_splits >= 1, "moe_combine: an addend of %d slices", also_splits);
     if (rows == 0) return 0;
@@ -497,7 +511,7 @@ extern "C" int kb_moe_combine(void* out, int out_dt, const float* y, const float
     KB_REQUIRE(blocks <= 0x7fffffffll, "moe_combine: too many rows for one launch");
     cudaStream_t s = (cudaStream_t)stream;
 #define KB_COMBINE(TO, TA) \
-    moe_combine_kernel<TO, TA><<<(unsigned)blocks, 256, 0, s>>>((TO*)out, y, weights, rows, width, top, Src<TA>{(const TA*)also, also ? also_splits : 1, (size_t)also_stride})
+    moe_combine_kernel<TO, TA><<<(unsigned)blocks, 256, 0, s>>>((TO*)out, y, weights, rows, width, top, Src<TA>{(const TA*)also, also ? also_splits : 1, (size_t)also_stride}, experts, real, self, self_dt)
     const bool narrow = also != nullptr && also_dt == KB_DT_BF16;
     KB_REQUIRE(also == nullptr || also_dt == KB_DT_F32 || also_dt == KB_DT_BF16, "moe_combine: addend dtype code %d is not known", also_dt);
     if (out_dt == KB_DT_F32) { if (narrow) KB_COMBINE(float, bf16); else KB_COMBINE(float, float); }

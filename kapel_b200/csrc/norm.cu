@@ -503,12 +503,12 @@ __global__ void add_rmsnorm_splits_bulk_kernel(float* __restrict__ residual, con
 }
 
 // ---------------------------------------------------------------------------------------
-// Norms that may take the mean off first (a layer norm with a weight and no bias):
-// y = (x - mean) / sqrt(mean((x - mean)^2) + eps) * (offset + w); without `center` the RMS norm above.
+// Norms that may take the mean off first (a layer norm with a weight, alone also with a bias):
+// y = (x - mean) / sqrt(mean((x - mean)^2) + eps) * (offset + w) + bias; without `center` the RMS norm above.
 // The variance is the mean of the squared deviations, taken in a second walk over the row.
 template <typename TX, typename TW, typename TY>
-__global__ void centered_norm_kernel(TY* __restrict__ y, const TX* __restrict__ x, const TW* __restrict__ w, int width,
-                                     float eps, float offset) {
+__global__ void centered_norm_kernel(TY* __restrict__ y, const TX* __restrict__ x, const TW* __restrict__ w, const TW* __restrict__ bias,
+                                     int width, float eps, float offset) {
     __shared__ float scratch[32];
     const size_t base = (size_t)blockIdx.x * width;
     float sum = 0.f;
@@ -523,7 +523,7 @@ __global__ void centered_norm_kernel(TY* __restrict__ y, const TX* __restrict__ 
     const float inv = 1.f / sqrtf(ss / (float)width + eps);
     for (int i = threadIdx.x; i < width; i += blockDim.x) {
         const float v = Elem<TX>::load(x + base + i) - mean;
-        Elem<TY>::store(y + base + i, v * inv * (offset + Elem<TW>::load(w + i)));
+        Elem<TY>::store(y + base + i, v * inv * (offset + Elem<TW>::load(w + i)) + (bias != nullptr ? Elem<TW>::load(bias + i) : 0.f));
     }
 }
 
@@ -731,8 +731,8 @@ extern "C" int kb_add_rmsnorm(float* residual, const void* branch, int branch_dt
 }
 
 
-// The centered norm alone. x: f32 or bf16; w: f32 or bf16; y: f32 or bf16.
-extern "C" int kb_layernorm(void* y, int y_dt, const void* x, int x_dt, const void* w, int w_dt, int rows, int width,
+// The centered norm alone. x: f32 or bf16; w and bias (or null): f32 or bf16; y: f32 or bf16.
+extern "C" int kb_layernorm(void* y, int y_dt, const void* x, int x_dt, const void* w, const void* bias, int w_dt, int rows, int width,
                             float eps, float offset, void* stream) {
     KB_REQUIRE(rows >= 0 && width > 0, "layernorm: rows %d, width %d", rows, width);
     KB_REQUIRE(eps >= 0.f, "layernorm: eps %g is negative", eps);
@@ -740,7 +740,7 @@ extern "C" int kb_layernorm(void* y, int y_dt, const void* x, int x_dt, const vo
     cudaStream_t s = (cudaStream_t)stream;
     const int t = threads_for(width);
 #define KB_LNORM(TX, TW, TY) \
-    centered_norm_kernel<TX, TW, TY><<<rows, t, 0, s>>>((TY*)y, (const TX*)x, (const TW*)w, width, eps, offset)
+    centered_norm_kernel<TX, TW, TY><<<rows, t, 0, s>>>((TY*)y, (const TX*)x, (const TW*)w, (const TW*)bias, width, eps, offset)
     const int code = x_dt * 4 + w_dt * 2 + y_dt;
     switch (code) {
         case 0: KB_LNORM(float, float, float); break;

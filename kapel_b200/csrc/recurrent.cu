@@ -419,10 +419,11 @@ struct RetentionParams {
     const float2* cos_sin;      // [rows, rotary / 2]
     int rotary, heads, d, e;
     float k_scale;
+    int act;                    // 1: silu on queries, keys and values as they come from the product
 };
 
-// One block a row, a warp a head: queries and keys turned (component i with i + rotary / 2), keys scaled; the scan's inputs
-// are decay q and k.
+// One block a row, a warp a head: queries, keys and values through the activation, queries and keys turned (component i with
+// i + rotary / 2), keys scaled; the scan's inputs are decay q and k.
 template <typename TS>
 __global__ void __launch_bounds__(256)
 retention_prep_kernel(const Src<TS> src, const RetentionParams p, const ScanInputs s) {
@@ -430,6 +431,10 @@ retention_prep_kernel(const Src<TS> src, const RetentionParams p, const ScanInpu
     const size_t base = (size_t)r * p.row_width;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, warps = blockDim.x >> 5;
     const int half = p.rotary >> 1, d = p.d;
+    auto at = [&](size_t i) {
+        const float v = src.at(i);
+        return p.act == 1 ? v * rc_sigmoid(v) : v;
+    };
     for (int h = warp; h < p.heads; h += warps) {
         float kr = 0.f;
         const float decay = p.decay[h];
@@ -442,14 +447,14 @@ retention_prep_kernel(const Src<TS> src, const RetentionParams p, const ScanInpu
         };
         const size_t qa = base + p.q_off + (size_t)h * d, ka = base + p.k_off + (size_t)h * d;
         for (int i = lane; i < half; i += 32) {
-            float q0 = src.at(qa + i), q1 = src.at(qa + half + i), k0 = src.at(ka + i), k1 = src.at(ka + half + i);
+            float q0 = at(qa + i), q1 = at(qa + half + i), k0 = at(ka + i), k1 = at(ka + half + i);
             const float2 cs = p.cos_sin[(size_t)r * half + i];
             rope_rotate(q0, q1, cs);
             rope_rotate(k0, k1, cs);
             put(i, q0, k0);
             put(half + i, q1, k1);
         }
-        for (int i = 2 * half + lane; i < d; i += 32) put(i, src.at(qa + i), src.at(ka + i));
+        for (int i = 2 * half + lane; i < d; i += 32) put(i, at(qa + i), at(ka + i));
         kr = warp_sum(kr);
         if (lane == 0) {
             s.scal[((size_t)r * p.heads + h) * 2] = 0.f;
@@ -457,7 +462,7 @@ retention_prep_kernel(const Src<TS> src, const RetentionParams p, const ScanInpu
         }
     }
     const int nv = p.heads * p.e;
-    for (int i = threadIdx.x; i < nv; i += blockDim.x) s.val[(size_t)r * nv + i] = src.at(base + p.v_off + i);
+    for (int i = threadIdx.x; i < nv; i += blockDim.x) s.val[(size_t)r * nv + i] = at(base + p.v_off + i);
 }
 
 // ------------------------------------------------------------------------------------------ the scan
@@ -959,7 +964,7 @@ extern "C" long long kb_retention_scratch_floats(int rows, int entries, int long
 // The read-out [rows, heads, e] of a matrix memory with a fixed decay a head behind rotated queries and keys. `longest`: the
 // most rows a request brings (every request's rows lie behind the earlier requests').
 extern "C" int kb_retention_scan(float* out, float* scratch, const void* src, int in_dt, int splits, long long split_stride, int row_width,
-                                 int q_off, int k_off, int v_off, const float* decay, const float* cos_sin, int rotary, float k_scale,
+                                 int q_off, int k_off, int v_off, const float* decay, const float* cos_sin, int rotary, float k_scale, int act,
                                  float* state, int n_slots, const int* entry_start, const int* entry_end, const int* slots, int entries,
                                  int rows, int longest, int heads, int d, int e, void* stream) {
     if (int err = scan_common_checks("retention", src, splits, split_stride, row_width, rows, entries, heads, d, e, state, n_slots, entry_start, entry_end, slots))
@@ -969,10 +974,11 @@ extern "C" int kb_retention_scan(float* out, float* scratch, const void* src, in
                "retention: columns q %d, k %d, v %d do not fit a row of %d", q_off, k_off, v_off, row_width);
     KB_REQUIRE(rotary >= 0 && rotary <= d && rotary % 2 == 0 && (rotary == 0 || cos_sin), "retention: a rotation of %d components of %d", rotary, d);
     KB_REQUIRE(out && scratch && decay, "retention: decays or scratch are missing");
+    KB_REQUIRE(act == 0 || act == 1, "retention: activation code %d is not known (0 none, 1 silu)", act);
     if (entries == 0 || rows == 0) return 0;
     RetentionParams g;
     g.row_width = row_width; g.q_off = q_off; g.k_off = k_off; g.v_off = v_off; g.decay = decay; g.cos_sin = (const float2*)cos_sin;
-    g.rotary = rotary; g.heads = heads; g.d = d; g.e = e; g.k_scale = k_scale;
+    g.rotary = rotary; g.heads = heads; g.d = d; g.e = e; g.k_scale = k_scale; g.act = act;
     ScanInputs in;
     in.vec = scratch;
     in.val = in.vec + (size_t)rows * nq * 2;

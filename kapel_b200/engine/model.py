@@ -30,6 +30,9 @@ class ModelParts:
             if e.before is not None and e.before not in self.merges:
                 self.merges[e.before] = build_part("merge", e.before, ctx)
         self.tap = None                                    # a function (run, residual) called after every layer run, for inspection
+        self.streams = int(spec.streams)
+        if any((layer.streams is not None) != bool(self.streams) for layer in spec.layers) or (self.streams and self.merges):
+            raise ValueError("a model of several residual streams has layers of kind \"streams\" and nothing that rewrites the stream between them")
         self.final_norm = build_part("norm", spec.final_norm, ctx)
         self.head = build_part("head", spec.head, ctx)
 
@@ -43,6 +46,8 @@ class ModelParts:
         for m in self.merges.values():
             m.load(tensors)
         self.final_norm.load(tensors)
+        if getattr(self.spec.head, "scale", 1.0) != 1.0:
+            self.final_norm.scale_output(float(self.spec.head.scale))  # the logits' scale goes in with the norm, in 32-bit
         self.head.load(tensors)
 
     def graph_safe(self) -> bool:
@@ -59,10 +64,11 @@ class ModelParts:
 
     def forward(self, batch, cache_manager) -> torch.Tensor:
         """float32 logits [wanted rows, vocab] of a step."""
+        copies = {"copies": self.streams} if self.streams else {}
         if getattr(self.embedding, "needs_positions", False):
-            x = self.embedding.forward(batch.ids, batch.positions)
+            x = self.embedding.forward(batch.ids, batch.positions, **copies)
         else:
-            x = self.embedding.forward(batch.ids)
+            x = self.embedding.forward(batch.ids, **copies)
         schedule = self.spec.schedule
         x0 = None
         if self.merges:
@@ -79,5 +85,5 @@ class ModelParts:
             x, h = block.forward(x, h, batch, cache, nxt)
             if self.tap is not None:
                 self.tap(i, x)
-        rows = K.gather_rows(x, batch.want_rows)
+        rows = K.stream_sum(x, self.streams, batch.want_rows) if self.streams else K.gather_rows(x, batch.want_rows)
         return self.head.forward(self.final_norm.forward(rows))

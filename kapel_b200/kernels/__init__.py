@@ -20,6 +20,7 @@ F32, BF16 = 0, 1
 _CODES = {torch.float32: F32, torch.bfloat16: BF16}
 
 ACT_CODES = {"gelu_tanh": 0, "silu": 1}
+GLU_EPILOGUES = {**ACT_CODES, "clamped_swish": 2}        # the gated units that a product's epilogue applies
 
 # Which kernel multiplies more than 64 rows of bfloat16: "tcgen05" (TMA, TMEM, tcgen05.mma; the
 # library picks between one block a tile and persistent pairs of blocks, "single" and "pair" force
@@ -228,8 +229,29 @@ class SplitSum:
         return self.partials.device
 
 
+class NormedSum:
+    """Two branches [rows, width] (tensors or SplitSums), each RMS-normed and weighted channel by channel, then added:
+    rms(a) weight_a + rms(b) weight_b (float32 weights). The kernel that adds branches to several streams norms them on
+    the way in; for anything else `finish` makes the sum."""
+
+    __slots__ = ("a", "b", "weight_a", "weight_b", "eps")
+
+    def __init__(self, a, weight_a: torch.Tensor, b, weight_b: torch.Tensor, eps: float):
+        self.a, self.weight_a, self.b, self.weight_b, self.eps = a, weight_a, b, weight_b, float(eps)
+
+    @property
+    def shape(self):
+        return tuple(self.a.shape)
+
+    @property
+    def device(self):
+        return self.a.device
+
+
 def _src(x, what: str):
-    """(tensor to read, dtype code, slices, elements between slices) of a tensor or a SplitSum."""
+    """(tensor to read, dtype code, slices, elements between slices) of a tensor, a SplitSum or a NormedSum."""
+    if isinstance(x, NormedSum):
+        x = finish(x, torch.float32)
     if isinstance(x, SplitSum):
         t = _need(x.partials, what, torch.float32)
         return t, F32, x.splits, t.shape[1] * t.shape[2]
@@ -238,7 +260,11 @@ def _src(x, what: str):
 
 
 def finish(x, dtype: torch.dtype) -> torch.Tensor:
-    """A SplitSum added up into a tensor of `dtype`; a tensor as it is (cast if need be)."""
+    """A SplitSum or a NormedSum added up into a tensor of `dtype`; a tensor as it is (cast if need be)."""
+    if isinstance(x, NormedSum):
+        total = rmsnorm(finish(x.a, torch.float32), x.weight_a, x.eps, 0.0, torch.float32)
+        add_rmsnorm(total, rmsnorm(finish(x.b, torch.float32), x.weight_b, x.eps, 0.0, torch.float32), None, None, torch.float32)
+        return total if dtype == torch.float32 else cast(total, dtype)
     if isinstance(x, SplitSum):
         _need(x.partials, "finish partials", torch.float32)
         out = _fresh(x.shape, dtype, x.device)
@@ -250,9 +276,9 @@ def finish(x, dtype: torch.dtype) -> torch.Tensor:
 
 # ------------------------------------------------------------------------------------------
 def embed(table: torch.Tensor, ids: torch.Tensor, scale: float, out: Optional[torch.Tensor] = None,
-          pos_table: Optional[torch.Tensor] = None, positions: Optional[torch.Tensor] = None) -> torch.Tensor:
+          pos_table: Optional[torch.Tensor] = None, positions: Optional[torch.Tensor] = None, copies: int = 1) -> torch.Tensor:
     """out[r] = table[ids[r]] * scale in float32; with `pos_table` [max positions, width] (the
-    table's dtype) and the rows' `positions`, plus pos_table[positions[r]] (not scaled)."""
+    table's dtype) and the rows' `positions`, plus pos_table[positions[r]] (not scaled). The row `copies` times side by side."""
     _need(table, "embed table")
     _need(ids, "embed ids", torch.int32)
     vocab, width = table.shape
@@ -265,10 +291,10 @@ def embed(table: torch.Tensor, ids: torch.Tensor, scale: float, out: Optional[to
         _need(positions, "embed positions", torch.int32, (rows,))
         most = int(pos_table.shape[0])
     if out is None:
-        out = _fresh((rows, width), torch.float32, table.device)
-    _need(out, "embed out", torch.float32, (rows, width))
+        out = _fresh((rows, copies * width), torch.float32, table.device)
+    _need(out, "embed out", torch.float32, (rows, copies * width))
     _check(library().kb_embed(_ptr(out), _ptr(table), _dt(table, "embed table"), _ptr(ids), rows, width, vocab, _f(scale),
-                              _ptr(pos_table), _ptr(positions if pos_table is not None else None), most, _stream()))
+                              _ptr(pos_table), _ptr(positions if pos_table is not None else None), most, int(copies), _stream()))
     return out
 
 
@@ -421,14 +447,17 @@ def rmsnorm(x: torch.Tensor, weight: torch.Tensor, eps: float, offset: float, ou
     return y
 
 
-def layernorm(x: torch.Tensor, weight: torch.Tensor, eps: float, offset: float, out_dtype: torch.dtype) -> torch.Tensor:
-    """(x - mean) / sqrt(mean((x - mean)^2) + eps) * (offset + weight) over each row, in 32-bit."""
+def layernorm(x: torch.Tensor, weight: torch.Tensor, eps: float, offset: float, out_dtype: torch.dtype,
+              bias: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """(x - mean) / sqrt(mean((x - mean)^2) + eps) * (offset + weight) + bias over each row, in 32-bit."""
     _need(x, "layernorm input")
     rows, width = x.shape
     _need(weight, "layernorm weight", shape=(width,))
+    if bias is not None:
+        _need(bias, "layernorm bias", weight.dtype, (width,))
     y = _fresh((rows, width), out_dtype, x.device)
     _check(
-        library().kb_layernorm(_ptr(y), _dt(y, "layernorm output"), _ptr(x), _dt(x, "layernorm input"), _ptr(weight),
+        library().kb_layernorm(_ptr(y), _dt(y, "layernorm output"), _ptr(x), _dt(x, "layernorm input"), _ptr(weight), _ptr(bias),
                                _dt(weight, "layernorm weight"), rows, width, _f(eps), _f(offset), _stream())
     )
     return y
@@ -561,16 +590,17 @@ def gemm(a: torch.Tensor, w: torch.Tensor, out_dtype: Optional[torch.dtype] = No
 _TCGEN05_KERNELS = {"tcgen05": 0, "single": 1, "pair": 2}       # the kernel chooses; one block a tile; persistent pairs
 
 
-def gemm_glu_fused(a: torch.Tensor, w: torch.Tensor, act: str) -> Optional[torch.Tensor]:
+def gemm_glu_fused(a: torch.Tensor, w: torch.Tensor, act: str, limit: float = 0.0, alpha: float = 0.0) -> Optional[torch.Tensor]:
     """act(a . gate^T) * (a . up^T) for a stacked gate|up weight w [2 n, k], in one kernel whose
     epilogue applies the gated unit to the 32-bit sums; None where no such kernel applies
-    (32-bit operands, the mma.sync yardsticks selected) and the caller multiplies and gates in two steps."""
+    (32-bit operands, the mma.sync yardsticks selected) and the caller multiplies and gates in two steps. The activation
+    "clamped_swish" is the bounded unit of `glu_clamped`."""
     if a.dtype != torch.bfloat16 or w.dtype != torch.bfloat16 or a.shape[0] == 0:
         return None
     few = a.shape[0] <= 64
     if (few and GEMM_SMALL != "skinny") or (not few and GEMM_LARGE not in ("tcgen05", "pair")):
         return None
-    if act not in ACT_CODES:
+    if act not in GLU_EPILOGUES:
         raise KernelError(f"gemm_glu: activation {act!r} is not known")
     _need(a, "gemm input")
     _need(w, "gemm weight")
@@ -580,9 +610,9 @@ def gemm_glu_fused(a: torch.Tensor, w: torch.Tensor, act: str) -> Optional[torch
         raise KernelError(f"gemm_glu: input [{m}, {k}] against stacked weight [{n2}, {k2}]")
     out = _fresh((m, n2 // 2), torch.bfloat16, a.device)
     if few:
-        _check(library().kb_gemm_skinny_glu(_ptr(out), _ptr(a), _ptr(w), m, n2 // 2, k, ACT_CODES[act], _stream()))
+        _check(library().kb_gemm_skinny_glu(_ptr(out), _ptr(a), _ptr(w), m, n2 // 2, k, GLU_EPILOGUES[act], _f(limit), _f(alpha), _stream()))
         return out
-    _check(library().kb_gemm_tcgen05_glu(_ptr(out), _ptr(a), _ptr(w), m, n2 // 2, k, ACT_CODES[act], _stream()))
+    _check(library().kb_gemm_tcgen05_glu(_ptr(out), _ptr(a), _ptr(w), m, n2 // 2, k, GLU_EPILOGUES[act], _f(limit), _f(alpha), _stream()))
     return out
 
 
@@ -1313,14 +1343,20 @@ def cdelta_scan(stacked, q_off: int, b_off: int, a1_off: int, a2: torch.Tensor, 
     return out
 
 
+RETENTION_ACTS = {"none": 0, "silu": 1}
+
+
 def retention_scan(stacked, q_off: int, k_off: int, v_off: int, decay: torch.Tensor, cos_sin, rotary: int, k_scale: float,
-                   state: torch.Tensor, ranges, slots, entries: int, longest: int, heads: int, d: int, e: int) -> torch.Tensor:
+                   state: torch.Tensor, ranges, slots, entries: int, longest: int, heads: int, d: int, e: int,
+                   act: str = "none") -> torch.Tensor:
     """The read-out [rows, heads, e] (float32, not yet normed) of a matrix memory with a fixed decay a head
-    (`decay` [heads]): S <- decay S + k v^T, o = S^T q, queries and keys turned by `cos_sin` [rows, rotary/2, 2]
+    (`decay` [heads]): S <- decay S + k v^T, o = S^T q; queries, keys and values through `act` ("none" or "silu"), queries and keys turned by `cos_sin` [rows, rotary/2, 2]
     (component i with i + rotary/2), keys then times `k_scale`; `state` [slots, heads e d]. `longest`: the most rows
     a request brings; a long portion is walked by chunks of rows (`retention_chunk_rows`)."""
     src, dt, splits, stride, rows, width = _stacked(stacked, "retention input")
     _need(decay, "retention decays", torch.float32, (heads,))
+    if act not in RETENTION_ACTS:
+        raise KernelError(f"retention: activation {act!r} is not known ({sorted(RETENTION_ACTS)})")
     if rotary:
         _need(cos_sin, "retention cos_sin", torch.float32, (rows, rotary // 2, 2))
     _need(state, "retention state", torch.float32)
@@ -1331,7 +1367,7 @@ def retention_scan(stacked, q_off: int, k_off: int, v_off: int, decay: torch.Ten
     scratch = _fresh((max(1, int(library().kb_retention_scratch_floats(rows, int(entries), int(longest), heads, d, e))),), torch.float32, src.device)
     _check(library().kb_retention_scan(
         _ptr(out), _ptr(scratch), _ptr(src), dt, splits, ctypes.c_longlong(stride), width, int(q_off), int(k_off), int(v_off), _ptr(decay),
-        _ptr(cos_sin if rotary else None), int(rotary), _f(k_scale), _ptr(state), int(state.shape[0]), _ptr(start), _ptr(end), _ptr(slots),
+        _ptr(cos_sin if rotary else None), int(rotary), _f(k_scale), RETENTION_ACTS[act], _ptr(state), int(state.shape[0]), _ptr(start), _ptr(end), _ptr(slots),
         int(entries), rows, int(longest), int(heads), int(d), int(e), _stream()))
     return out
 
@@ -1420,7 +1456,7 @@ def proj_rope_append(stacked, q_off: int, k_off: int, v_off: int, biases, q_norm
     `biases[0]`, normed over the whole projection when `q_norm` = (weight [hq d], eps, offset) is given,
     the first `rotary` components of every head turned by `cos_sin` [rows, rotary/2, 2] (pairs
     (i, i + rotary/2), or (2i, 2i+1) with `neighbours`). Keys likewise (`biases[1]`, `k_norm`) and written
-    at each row's line of the table [pages, hkv, page_size, d]. Values: plus `biases[2]`; with `v_other`
+    at each row's line of the table [pages, hkv, page_size, d] (`hkv` 0: queries alone). Values: plus `biases[2]`; with `v_other`
     [rows, hkv dv] float32 and `v_weight` (one value l on the device) v <- (1 - l) v + l v_other; written
     to the table [.., dv]. Returns (q, the values before that mix as float32 [rows, hkv dv] if
     `keep_values`, else None). Biases and norm weights share a dtype."""
@@ -1582,9 +1618,9 @@ ROUTE_SCORING = {"sigmoid": 0, "softmax": 1, "softmax_chosen": 2}
 
 
 def moe_route(h: torch.Tensor, router: torch.Tensor, correction: Optional[torch.Tensor], top: int, groups: int, keep_groups: int,
-              group_top: int, scoring: str, renormalize: bool):
+              group_top: int, scoring: str, renormalize: bool, scale: float = 1.0):
     """(experts int32 [rows, top], weights float32 [rows, top]) of each row of h [rows, width];
-    the router [experts, width] and the correction [experts] are float32."""
+    the router [experts, width] and the correction [experts] are float32. The weights are multiplied by `scale` at the end."""
     _need(h, "moe_route input")
     rows, width = h.shape
     _need(router, "moe_route router", torch.float32)
@@ -1599,7 +1635,7 @@ def moe_route(h: torch.Tensor, router: torch.Tensor, correction: Optional[torch.
     weights = _fresh((rows, top), torch.float32, h.device)
     _check(library().kb_moe_route(_ptr(experts), _ptr(weights), _ptr(h), _dt(h, "moe_route input"), _ptr(router), _ptr(correction),
                                   rows, width, n_experts, int(top), int(groups), int(keep_groups), int(group_top),
-                                  ROUTE_SCORING[scoring], int(bool(renormalize)), _stream()))
+                                  ROUTE_SCORING[scoring], int(bool(renormalize)), _f(scale), _stream()))
     return experts, weights
 
 
@@ -1610,7 +1646,7 @@ class ExpertLists:
 
 
 def moe_sort(experts: torch.Tensor, n_experts: int, dtype: torch.dtype = torch.float32) -> ExpertLists:
-    """Lists the pairs of `experts` [rows, top] by expert; `dtype` is the grouped products' (it and the
+    """Lists the pairs of `experts` [rows, top] by expert, those from number `n_experts` on (experts without weights) left out; `dtype` is the grouped products' (it and the
     rows an expert gets on average decide how many rows a tile of those products has)."""
     _need(experts, "moe_sort experts", torch.int32)
     rows, top = experts.shape
@@ -1652,9 +1688,11 @@ def moe_grouped(a: torch.Tensor, w: torch.Tensor, lists: ExpertLists, act: str, 
     return out
 
 
-def moe_combine(y: torch.Tensor, weights: torch.Tensor, out_dtype: torch.dtype, also=None) -> torch.Tensor:
+def moe_combine(y: torch.Tensor, weights: torch.Tensor, out_dtype: torch.dtype, also=None, experts: Optional[torch.Tensor] = None,
+                real: int = 0, own: Optional[torch.Tensor] = None) -> torch.Tensor:
     """out[token] = sum over k, in order, of weights[token, k] * y[token * top + k], plus `also`[token]
-    where given (a tensor or a SplitSum [tokens, width]: the output of an expert that every token uses)."""
+    where given (a tensor or a SplitSum [tokens, width]: the output of an expert that every token uses). With `experts`
+    [tokens, top], a pair whose expert's number is `real` or more takes the token's row of `own` [tokens, width] in place of y's."""
     _need(y, "moe_combine input", torch.float32)
     _need(weights, "moe_combine weights", torch.float32)
     rows, top = weights.shape
@@ -1666,9 +1704,78 @@ def moe_combine(y: torch.Tensor, weights: torch.Tensor, out_dtype: torch.dtype, 
         a_src, a_dt, a_splits, a_stride = _src(also, "moe_combine addend")
         if tuple(also.shape) != (rows, width):
             raise KernelError(f"moe_combine: an addend {tuple(also.shape)} beside a sum of {(rows, width)}")
+    if (experts is None) != (own is None):
+        raise KernelError("moe_combine: identity experts and the rows they give back come together")
+    if experts is not None:
+        _need(experts, "moe_combine experts", torch.int32, (rows, top))
+        _need(own, "moe_combine own rows", shape=(rows, width))
     out = _fresh((rows, width), out_dtype, y.device)
     _check(library().kb_moe_combine(_ptr(out), _CODES[out_dtype], _ptr(y), _ptr(weights), ctypes.c_longlong(rows), int(width), int(top),
-                                    _ptr(a_src), a_dt, int(a_splits), ctypes.c_longlong(a_stride), _stream()))
+                                    _ptr(a_src), a_dt, int(a_splits), ctypes.c_longlong(a_stride), _ptr(experts), int(real), _ptr(own),
+                                    _dt(own, "moe_combine own rows") if own is not None else F32, _stream()))
+    return out
+
+
+# ------------------------------------------------------------------------------------------
+# Several residual streams a row (hyper-connections).
+def stream_step(x: torch.Tensor, streams: int, write=None, read=None, out_dtype: Optional[torch.dtype] = None) -> Optional[torch.Tensor]:
+    """One row's streams x [rows, streams * width] (float32, updated in place) between two sublayers. `write` = (branch, a
+    weight a channel [width] or None, mix [streams, streams], out [streams]): x_t <- sum_s mix[s, t] x_s + out[t] branch * weight,
+    all streams from the old ones. `read` = (in [streams], norm weight [width], bias [width] or None, eps, offset, center):
+    returns norm(sum_s in[s] x_s) in `out_dtype`, a layer norm with `center`, else an RMS norm. Everything but
+    the branch (a tensor, a SplitSum or a NormedSum) and the result is float32."""
+    _need(x, "stream_step streams", torch.float32)
+    rows, all_widths = x.shape
+    if streams < 1 or all_widths % streams:
+        raise KernelError(f"stream_step: rows of {all_widths} values in {streams} streams")
+    width = all_widths // streams
+    a_src = b_src = scale = mix = out = n_a = n_b = None
+    dt, a_splits, a_stride, b_splits, b_stride, eps_ab = F32, 1, 0, 1, 0, 0.0
+    if write is not None:
+        branch, scale, mix, out = write
+        if tuple(branch.shape) != (rows, width):
+            raise KernelError(f"stream_step: a branch {tuple(branch.shape)} against streams of {(rows, width)}")
+        _need(mix, "stream_step mix", torch.float32, (streams, streams))
+        _need(out, "stream_step out", torch.float32, (streams,))
+        if scale is not None:
+            _need(scale, "stream_step branch weights", torch.float32, (width,))
+        if isinstance(branch, NormedSum):
+            a_src, dt, a_splits, a_stride = _src(branch.a, "stream_step first branch")
+            b_src, b_dt, b_splits, b_stride = _src(branch.b, "stream_step second branch")
+            if tuple(branch.b.shape) != (rows, width) or b_dt != dt:
+                raise KernelError(f"stream_step: branches {tuple(branch.a.shape)} and {tuple(branch.b.shape)} of one shape and dtype are needed")
+            n_a = _need(branch.weight_a, "stream_step first norm", torch.float32, (width,))
+            n_b = _need(branch.weight_b, "stream_step second norm", torch.float32, (width,))
+            eps_ab = branch.eps
+        else:
+            a_src, dt, a_splits, a_stride = _src(branch, "stream_step branch")
+    h = w_in = weight = bias = None
+    eps, offset, center = 0.0, 0.0, False
+    if read is not None:
+        w_in, weight, bias, eps, offset, center = read
+        _need(w_in, "stream_step in", torch.float32, (streams,))
+        _need(weight, "stream_step norm", torch.float32, (width,))
+        if bias is not None:
+            _need(bias, "stream_step norm bias", torch.float32, (width,))
+        h = _fresh((rows, width), out_dtype or torch.float32, x.device)
+    _check(library().kb_stream_step(
+        _ptr(x), int(rows), int(streams), int(width), _ptr(a_src), int(a_splits), ctypes.c_longlong(a_stride), _ptr(b_src), int(b_splits),
+        ctypes.c_longlong(b_stride), dt, _ptr(n_a), _ptr(n_b), _f(eps_ab), _ptr(scale), _ptr(mix), _ptr(out), _ptr(w_in),
+        _ptr(weight), _ptr(bias), _f(eps), _f(offset), int(bool(center)), _ptr(h), _dt(h, "stream_step output") if h is not None else F32, _stream()))
+    return h
+
+
+def stream_sum(x: torch.Tensor, streams: int, rows: torch.Tensor) -> torch.Tensor:
+    """The streams of the rows `rows` (int32 on the device) of x [all rows, streams * width], added up: float32 [n, width]."""
+    _need(x, "stream_sum streams", torch.float32)
+    _need(rows, "stream_sum rows", torch.int32)
+    if streams < 1 or x.shape[1] % streams:
+        raise KernelError(f"stream_sum: rows of {x.shape[1]} values in {streams} streams")
+    width, n = x.shape[1] // streams, rows.numel()
+    out = _fresh((n, width), torch.float32, x.device)
+    for at in range(0, n, 65535):
+        m = min(65535, n - at)
+        _check(library().kb_stream_sum(_ptr(out[at:]), _ptr(x), _ptr(rows[at:]), int(m), int(width), int(streams), int(x.shape[0]), _stream()))
     return out
 
 
@@ -1697,7 +1804,7 @@ _TIMED = ("embed", "rope_table", "rope_append", "glu", "cast", "gather_rows", "r
           "moe_sort", "moe_grouped", "moe_combine", "gemm_glu_fused", "paged_attention_decode_fused", "layernorm", "concat2",
           "head_norm_rope_append", "latent_append", "head_linear", "delta_scan", "latent_attention_mma", "proj_rope_append",
           "pool_blocks", "pooled_attention", "act", "token_shift", "conv_append", "gdelta_scan", "gate_scan", "weighted_sum2",
-          "glu_clamped", "cdelta_scan", "retention_scan", "conv_rows", "lru_gates", "lru_scan", "take_cols")
+          "glu_clamped", "stream_step", "stream_sum", "cdelta_scan", "retention_scan", "conv_rows", "lru_gates", "lru_scan", "take_cols")
 _timing = None
 _originals = {}
 

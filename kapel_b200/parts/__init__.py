@@ -18,6 +18,7 @@ from .parallel import ParallelMixer
 from .position import NoPosition, Rope
 from .retention import Retention
 from .rglru import RGLRU
+from .streams import StreamBlock
 from .registry import (
     build_part,
     part_class,
@@ -53,6 +54,7 @@ register_part("block", "sandwich", SandwichBlock)
 register_part("block", "prenorm", PreNormBlock)
 register_part("block", "postnorm", PostNormBlock)
 register_part("block", "parallel", ParallelBlock)
+register_part("block", "streams", StreamBlock)
 register_part("embedding", "embedding", Embedding)
 register_part("head", "vocab_head", VocabHead)
 

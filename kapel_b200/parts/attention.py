@@ -8,9 +8,11 @@ then the output product (model.rs:1633-1637).
 
 A spec may ask for more than that: a norm over the whole query and key projections, values of
 another size than keys, first keys that stay visible below the window, a sigmoid gate on the
-heads' outputs. Such a layer runs the general path: one stacked product q|k|v|g in 32-bit, one
-kernel that norms q and k and appends k and v to the cache, the row-wise attention kernel (which
-knows the kept first keys and the values' size), the gate, the output product.
+heads' outputs, a sink (learned, or 1 in the denominator) beside norms over the projection, keys and values that
+are another layer's. Such a layer runs the general path: one stacked product q|k|v|g in 32-bit (q|g where
+the keys are another layer's), one kernel that norms q and k, turns them (either pairing) and appends k and v to the
+cache, the tensor-core kernels where keys and values have one size and no first keys are kept (else the row-wise
+kernel), the gate, the output product.
 
 A spec with an RMS norm over every head's query and key (`q_head_norm`, `k_head_norm`: one weight
 of the head's size for all heads), a sink in the softmax's denominator or one gate a head runs the third
@@ -58,8 +60,9 @@ class Attention(Part):
             if spec.out_bias:
                 out[w["o_bias"]] = (spec.hidden,)
             return out
-        out = {w["q"]: (qd, spec.hidden), w["k"]: (kvd, spec.hidden), w["v"]: (spec.num_kv_heads * dv, spec.hidden),
-               w["o"]: (spec.hidden, spec.num_heads * dv)}
+        out = {w["q"]: (qd, spec.hidden), w["o"]: (spec.hidden, spec.num_heads * dv)}
+        if not spec.borrows_kv:
+            out[w["k"]], out[w["v"]] = (kvd, spec.hidden), (spec.num_kv_heads * dv, spec.hidden)
         if spec.gated:
             out[w["g"]] = (spec.num_heads if spec.gate_by_head else spec.num_heads * dv, spec.hidden)
         if spec.sink:
@@ -82,16 +85,17 @@ class Attention(Part):
         if spec.num_heads % spec.num_kv_heads:
             raise ValueError(f"attention: {spec.num_heads} heads over {spec.num_kv_heads} kv heads")
         self.v_dim = spec.v_head_dim or spec.head_dim
-        self.by_head = bool(spec.q_head_norm or spec.k_head_norm or spec.sink or spec.gate_by_head)
+        self.by_head = bool(spec.q_head_norm or spec.k_head_norm or spec.gate_by_head
+                            or (spec.sink and not (spec.q_norm or spec.k_norm or spec.borrows_kv)))
         if spec.gate_by_head and not spec.gated:
             raise ValueError("attention: one gate a head for a layer without a gate")
-        self.convolved = bool(spec.conv or spec.values_are_keys or spec.block_mask or spec.unit_sink or spec.qk_bias or spec.out_bias)
+        self.convolved = bool(spec.conv or spec.values_are_keys or spec.block_mask or spec.qk_bias or spec.out_bias)
         self.out_bias = None
         if self.convolved:
             if not (spec.values_are_keys and 1 <= spec.conv <= 16):
-                raise ValueError("attention: a block mask, 1 in the denominator or biases on q, k and o are built for the path with "
+                raise ValueError("attention: a block mask or biases on q, k and o are built for the path with "
                                  f"convolutions (1 to 16 rows, got {spec.conv}) whose values are its keys")
-            if (self.by_head or spec.gated or spec.q_norm or spec.k_norm or spec.keep_first or spec.softcap or spec.window or spec.bias
+            if (self.by_head or spec.borrows_kv or spec.gated or spec.q_norm or spec.k_norm or spec.keep_first or spec.softcap or spec.window or spec.bias
                     or spec.pool or spec.head_temp or spec.talk or spec.value_mix or spec.v_head_dim not in (None, spec.head_dim)):
                 raise ValueError("attention: convolutions together with norms, a sink, a gate, a window, a soft cap, pooled blocks, mixed heads or "
                                  "values of their own are not built")
@@ -99,18 +103,24 @@ class Attention(Part):
                 raise ValueError(f"attention: blocks of {spec.block_mask} positions")
         self.pooled = bool(spec.bias or spec.pool or spec.head_temp or spec.talk or spec.value_mix)
         if self.pooled:
-            if self.by_head or spec.gated or spec.keep_first or spec.softcap:
+            if self.by_head or spec.sink or spec.unit_sink or spec.borrows_kv or spec.gated or spec.keep_first or spec.softcap:
                 raise ValueError("attention: biases, pooled blocks, head temperatures, mixed heads or mixed values together with norms "
                                  "over each head, a sink, a gate, kept first keys or a soft cap are not built")
             if spec.pool and (not spec.window or spec.pool_blocks <= 0):
                 raise ValueError(f"attention: blocks of {spec.pool} need a window (got {spec.window}) and a count of blocks (got {spec.pool_blocks})")
             if spec.value_mix not in (None, "source", "mix"):
                 raise ValueError(f"attention: value_mix {spec.value_mix!r} is not known (\"source\", \"mix\")")
-        self.general = bool(spec.gated or spec.q_norm or spec.k_norm or spec.keep_first or self.v_dim != spec.head_dim) and not self.by_head \
-            and not self.pooled
-        if self.by_head and (spec.q_norm or spec.k_norm or spec.keep_first or spec.window):
-            raise ValueError("attention: norms over each head, a sink or one gate a head together with norms over the whole projection, a window "
-                             "or kept first keys are not built")
+        self.general = bool(spec.gated or spec.q_norm or spec.k_norm or spec.keep_first or self.v_dim != spec.head_dim or spec.borrows_kv
+                            or spec.unit_sink) and not self.by_head and not self.pooled and not self.convolved
+        if self.by_head and (spec.q_norm or spec.k_norm or spec.keep_first or spec.borrows_kv):
+            raise ValueError("attention: norms over each head or one gate a head together with norms over the whole projection, another layer's "
+                             "keys or kept first keys are not built")
+        if spec.sink and spec.unit_sink:
+            raise ValueError("attention: a learned sink and 1 in the denominator exclude one another")
+        if (spec.sink or spec.unit_sink) and spec.keep_first:
+            raise ValueError("attention: a sink together with kept first keys is not built")
+        if spec.borrows_kv and spec.k_norm:
+            raise ValueError("attention: a layer that takes another layer's keys has no norm of its own on them")
         for n in (spec.q_head_norm, spec.k_head_norm):
             if n is not None and (n.kind != "rms" or n.width != spec.head_dim):
                 raise ValueError(f"attention: a norm over each head must be an RMS norm of width {spec.head_dim}")
@@ -125,12 +135,11 @@ class Attention(Part):
             require_product_widths(ctx, "attention", hidden_size=spec.hidden,
                                    **{"num_attention_heads x value size": spec.num_heads * self.v_dim})
         self.position = build_part("position", spec.position, ctx)
-        if self.general and self.position.rotary_dim:
-            raise ValueError("attention: a rotation together with projection norms, a gate, kept first keys or another value size is not built")
         if self.convolved and self.position.rotary_dim:
             raise ValueError("attention: a rotation together with convolutions is not built")
-        if not self.pooled and getattr(self.position, "neighbours", False):
-            raise ValueError("attention: the rotation of neighbouring components is built for the path with biases, pooled blocks or mixed heads only")
+        if not self.pooled and not self.general and getattr(self.position, "neighbours", False):
+            raise ValueError("attention: the rotation of neighbouring components is built for the paths with biases, pooled blocks, mixed heads, "
+                             "norms over the projection or another layer's keys only")
 
     def load_convolved(self, tensors):
         s, w, dev = self.spec, self.spec.weights, self.ctx.device
@@ -150,22 +159,29 @@ class Attention(Part):
 
     def load_shared(self, tensors):
         """`load` without the two products' weights, for a caller that multiplies by them (`forward_stacked`)."""
+        self.load_sinks(tensors)
+        self.load_norms(tensors)
+
+    def load_sinks(self, tensors):
         s = self.spec
         self.sinks = tensors[s.weights["sink"]].to(self.ctx.device).float().contiguous() if s.sink else None
-        self.load_norms(tensors)
+        if s.unit_sink:
+            self.sinks = torch.zeros((s.num_heads,), dtype=torch.float32, device=self.ctx.device)       # e^0 = 1 in the denominator
 
     def load(self, tensors):
         if self.convolved:
             return self.load_convolved(tensors)
         w = self.spec.weights
-        names = [w["q"], w["k"], w["v"]] + ([w["g"]] if self.spec.gated else [])
+        names = [w["q"]] + ([] if self.spec.borrows_kv else [w["k"], w["v"]]) + ([w["g"]] if self.spec.gated else [])
         self.w_qkv = stack_rows(self.ctx, tensors, names, "attention")
         self.w_o = matrix_named(self.ctx, tensors, w["o"])
         if self.by_head:
             self.w_o = pad_columns(self.ctx, self.w_o)
             return self.load_shared(tensors)
-        if (self.general and self.spec.gated) or self.pooled:
+        if self.general or self.pooled:
             self.w_o = pad_columns(self.ctx, self.w_o)
+        if self.general:
+            self.load_sinks(tensors)
         if self.pooled:
             dev = self.ctx.device
             small = lambda name: (tensors[name].to(dev).float() if self.ctx.is_f32 else tensors[name].to(dev)).contiguous()
@@ -269,32 +285,43 @@ class Attention(Part):
 
     def forward_general(self, h, batch, cache):
         s, dv = self.spec, self.v_dim
-        nq, nk = s.num_heads * s.head_dim, s.num_kv_heads * s.head_dim
+        own = 0 if s.borrows_kv else s.num_kv_heads         # kv heads whose projections are in the product
+        nq, nk = s.num_heads * s.head_dim, own * s.head_dim
         stacked = linear(self.ctx, h, self.w_qkv, out_dtype=torch.float32, keep_split=True)
         k_table, v_table = cache.tables()
         group = batch.groups[cache.group]
-        q = K.proj_norm_append(stacked, 0, nq, nq + nk, self.proj_norms[0], self.proj_norms[1], group.lines, k_table, v_table,
-                               s.num_heads, s.num_kv_heads, s.head_dim, dv, cache.owns, self.ctx.dtype)
+        rotary = self.position.rotary_dim
+        if rotary or s.borrows_kv:
+            q, _ = K.proj_rope_append(
+                stacked, 0, nq, nq + nk, None, self.proj_norms[0], self.proj_norms[1], self.position.tables(batch) if rotary else None, rotary,
+                getattr(self.position, "neighbours", False), None, None, False, group.lines, k_table, v_table, s.num_heads, own, s.head_dim, dv,
+                cache.owns and own > 0, self.ctx.dtype)
+        else:
+            q = K.proj_norm_append(stacked, 0, nq, nq + nk, self.proj_norms[0], self.proj_norms[1], group.lines, k_table, v_table,
+                                   s.num_heads, s.num_kv_heads, s.head_dim, dv, cache.owns, self.ctx.dtype)
         heads_per_kv = s.num_heads // s.num_kv_heads
+        keep = s.keep_first if s.window else 0
         y = None
         if dv == s.head_dim and K.attention_mma_takes(q.dtype, s.head_dim, heads_per_kv):
-            # prompt portions go to the tensor-core kernel, which knows the kept first keys; a pass of
-            # single tokens stays with the row-wise kernel below
-            decode, tiles, split, slots, _ = batch.attention_tiles(heads_per_kv, s.num_kv_heads, s.window, s.head_dim, "mma",
-                                                                   keep_first=s.keep_first if s.window else 0)
-            if not decode:
+            # with kept first keys only prompt portions go to the tensor-core kernel; a pass of single tokens stays with
+            # the row-wise kernel below
+            prompt = "mma" if keep or self.sinks is not None else K.attention_prompt_kernel(s.num_heads, s.num_kv_heads, s.head_dim,
+                                                                                            self.ctx.page_size, s.softcap)
+            decode, tiles, split, slots, relative = batch.attention_tiles(heads_per_kv, s.num_kv_heads, s.window, s.head_dim, prompt, keep_first=keep)
+            if not (decode and keep):
                 y = K.paged_attention_mma(q, k_table, v_table, group.block_table, batch.row_count, tiles, self.ctx.page_size,
-                                          s.window, s.scale, s.softcap, 0, split, slots, False,
-                                          keep_first=s.keep_first if s.window else 0)
+                                          s.window, s.scale, s.softcap, decode, split, slots, relative, pairs=getattr(batch, "pairs", None),
+                                          keep_first=keep, sinks=self.sinks)
         if y is None:
             y = K.paged_attention_rows(
                 q, k_table, v_table, group.block_table, batch.row_entry, batch.row_count, self.ctx.page_size, s.window, s.scale,
-                s.softcap, batch.attention_slots(s.window, s.keep_first), s.keep_first)
+                s.softcap, batch.attention_slots(s.window, s.keep_first), s.keep_first, sinks=self.sinks)
+        width = product_width(self.ctx, s.num_heads * dv)
         if s.gated:
-            y = K.head_gate(y, stacked, nq + nk + s.num_kv_heads * dv, None, False, 0.0, self.ctx.dtype,
-                            pad_to=product_width(self.ctx, s.num_heads * dv))
+            y = K.head_gate(y, stacked, nq + nk + own * dv, None, False, 0.0, self.ctx.dtype, pad_to=width)
             return linear(self.ctx, y, self.w_o, keep_split=True)
-        return linear(self.ctx, y.view(y.shape[0], s.num_heads * dv), self.w_o, keep_split=True)
+        y = y.view(y.shape[0], s.num_heads * dv)
+        return linear(self.ctx, K.pad_cols(y, width) if width != y.shape[1] else y, self.w_o, keep_split=True)
 
     def forward_by_head(self, h, batch, cache):
         stacked = linear(self.ctx, h, self.w_qkv, out_dtype=torch.float32, keep_split=True)
@@ -319,12 +346,12 @@ class Attention(Part):
         heads_per_kv = s.num_heads // s.num_kv_heads
         if dv == s.head_dim and s.head_dim % 16 == 0 and K.attention_mma_takes(q.dtype, s.head_dim, heads_per_kv):
             prompt = "mma" if self.sinks is not None else K.attention_prompt_kernel(s.num_heads, s.num_kv_heads, s.head_dim, self.ctx.page_size, s.softcap)
-            decode, tiles, split, slots, relative = batch.attention_tiles(heads_per_kv, s.num_kv_heads, None, s.head_dim, prompt)
-            y = K.paged_attention_mma(q, k_table, v_table, group.block_table, batch.row_count, tiles, self.ctx.page_size, None,
+            decode, tiles, split, slots, relative = batch.attention_tiles(heads_per_kv, s.num_kv_heads, s.window, s.head_dim, prompt)
+            y = K.paged_attention_mma(q, k_table, v_table, group.block_table, batch.row_count, tiles, self.ctx.page_size, s.window,
                                       s.scale, s.softcap, decode, split, slots, relative, pairs=getattr(batch, "pairs", None), sinks=self.sinks)
         else:
             y = K.paged_attention_rows(q, k_table, v_table, group.block_table, batch.row_entry, batch.row_count, self.ctx.page_size,
-                                       None, s.scale, s.softcap, batch.attention_slots(None), sinks=self.sinks)
+                                       s.window, s.scale, s.softcap, batch.attention_slots(s.window), sinks=self.sinks)
         width = product_width(self.ctx, s.num_heads * dv) if pad_to is None else pad_to
         if s.gated or out is not None:
             return K.head_gate(y, stacked, base + nq + nk + s.num_kv_heads * dv if s.gated else 0, None, False, 0.0, self.ctx.dtype, pad_to=width,

@@ -39,12 +39,13 @@ class Embedding(Part):
             scale = float(torch.tensor(scale, dtype=torch.float32))
         self.scale = scale
 
-    def forward(self, ids, positions=None):
+    def forward(self, ids, positions=None, copies: int = 1):
+        """float32 [rows, copies x hidden]: a row's vector `copies` times side by side."""
         if self.pos_table is not None:
             if positions is None:
                 raise ValueError("embedding: a table of learned positions needs the rows' positions")
-            return K.embed(self.table, ids, self.scale, pos_table=self.pos_table, positions=positions)
-        return K.embed(self.table, ids, self.scale)
+            return K.embed(self.table, ids, self.scale, pos_table=self.pos_table, positions=positions, copies=copies)
+        return K.embed(self.table, ids, self.scale, copies=copies)
 
 
 class VocabHead(Part):

@@ -23,7 +23,10 @@ class GatedMLP(Part):
 
     def __init__(self, spec, ctx):
         super().__init__(spec, ctx)
-        if spec.activation not in K.ACT_CODES:
+        self.clamped = spec.activation == "clamped_swish"
+        if self.clamped and not (spec.limit is not None and spec.limit > 0):
+            raise ValueError(f"gated_mlp: the bounded gated unit needs a positive `limit`, got {spec.limit}")
+        if not self.clamped and spec.activation not in K.ACT_CODES:
             raise ValueError(f"gated_mlp: activation {spec.activation!r} is not built")
         # widths that are no multiple of 8 go through the products that pad their rows (`linear`), unfused
         self.fusable = spec.hidden % 8 == 0 and spec.intermediate % 8 == 0
@@ -35,10 +38,15 @@ class GatedMLP(Part):
 
     def forward(self, h):
         # many rows of bfloat16: the gated unit is the epilogue of the gate|up product
-        inner = K.gemm_glu_fused(h, self.w_gate_up, self.spec.activation) if (self.fusable and h.dtype == self.w_gate_up.dtype) else None
+        s, inner = self.spec, None
+        if self.fusable and h.dtype == self.w_gate_up.dtype:
+            inner = K.gemm_glu_fused(h, self.w_gate_up, s.activation, s.limit or 0.0, s.swish_alpha)
         if inner is None:
             gu = linear(self.ctx, h, self.w_gate_up, keep_split=True)
-            inner = K.glu(gu, self.spec.activation, out_dtype=self.ctx.dtype)
+            if self.clamped:
+                inner = K.glu_clamped(gu, s.limit, s.swish_alpha, out_dtype=self.ctx.dtype)
+            else:
+                inner = K.glu(gu, s.activation, out_dtype=self.ctx.dtype)
         return linear(self.ctx, inner, self.w_down, keep_split=True)
 
 

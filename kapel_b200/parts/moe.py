@@ -10,6 +10,8 @@ with this feed-forward can be recorded. All experts' weights of a role are one t
 (down(act(gate h) * up h)) keep gate and up of an expert one below the other: the first grouped
 product gives gate|up a pair, the gated unit's kernel the second product's input. A shared expert (a
 feed-forward part of its own that every token runs) is added in the kernel that sums the experts up.
+The router may have outputs beyond the experts: identity experts, which have no lists and no products; the
+last kernel adds the token's own input with their weight.
 The gated activation "clamped_swish" bounds both halves: min(gate, L) sigmoid(a min(gate, L)) (clamp(up, -L, L) + 1).
 """
 from __future__ import annotations
@@ -27,9 +29,9 @@ class MoE(Part):
     @staticmethod
     def expected_tensors(spec):
         w = spec.weights
-        out = {w["router"]: (spec.experts, spec.hidden)}
+        out = {w["router"]: (spec.experts + spec.identity, spec.hidden)}
         if w.get("correction"):
-            out[w["correction"]] = (spec.experts,)
+            out[w["correction"]] = (spec.experts + spec.identity,)
         for e in range(spec.experts):
             if spec.gated:
                 out[w["gate"].format(e=e)] = (spec.intermediate, spec.hidden)
@@ -49,10 +51,13 @@ class MoE(Part):
         if spec.scoring not in K.ROUTE_SCORING:
             raise ValueError(f"moe: scoring {spec.scoring!r} is not built")
         self.shared = build_part("feed_forward", spec.shared, ctx) if spec.shared is not None else None
-        if spec.experts % spec.groups or not 1 <= spec.keep_groups <= spec.groups:
-            raise ValueError(f"moe: {spec.experts} experts in {spec.groups} groups of which {spec.keep_groups} are kept")
-        if spec.keep_groups * (spec.experts // spec.groups) < spec.top or spec.top < 1:
-            raise ValueError(f"moe: {spec.keep_groups} groups of {spec.experts // spec.groups} experts cannot give {spec.top}")
+        if spec.identity < 0 or spec.experts < 1:
+            raise ValueError(f"moe: {spec.experts} experts and {spec.identity} identity experts")
+        outputs = spec.experts + spec.identity
+        if outputs % spec.groups or not 1 <= spec.keep_groups <= spec.groups:
+            raise ValueError(f"moe: {outputs} experts in {spec.groups} groups of which {spec.keep_groups} are kept")
+        if spec.keep_groups * (outputs // spec.groups) < spec.top or spec.top < 1:
+            raise ValueError(f"moe: {spec.keep_groups} groups of {outputs // spec.groups} experts cannot give {spec.top}")
 
     def load(self, tensors):
         s, w = self.spec, self.spec.weights
@@ -73,7 +78,8 @@ class MoE(Part):
     def forward(self, h):
         s = self.spec
         experts, weights = K.moe_route(h, self.router, self.correction, s.top, s.groups, s.keep_groups, s.group_top, s.scoring,
-                                       s.renormalize)
+                                       s.renormalize, s.route_scale)
+        own = h if s.identity else None
         lists = K.moe_sort(experts, s.experts, self.w_up.dtype)
         if h.dtype != self.w_up.dtype:
             h = K.cast(h, self.w_up.dtype)
@@ -87,4 +93,4 @@ class MoE(Part):
         else:
             inner = K.moe_grouped(h, self.w_up, lists, s.activation, True, False, self.w_up.dtype)
         y = K.moe_grouped(inner, self.w_down, lists, "none", False, True, torch.float32)
-        return K.moe_combine(y, weights, torch.float32, also=also)
+        return K.moe_combine(y, weights, torch.float32, also=also, experts=experts if s.identity else None, real=s.experts, own=own)
