@@ -377,7 +377,7 @@ gemm_tcgen05_pair_persistent_kernel(const __grid_constant__ CUtensorMap map_a, c
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     uint32_t rank;
     asm volatile("mov.u32 %0, %%cluster_ctarank;" : "=r"(rank));
-    constexpr bool glu = EPI == EPI_GLU_GELU || EPI == EPI_GLU_SILU;
+    constexpr bool glu = epi_glu(EPI);
     constexpr int tile_cols = glu ? TP_BN_HALF : 2 * TP_BN_HALF;
     const int m_pairs = (m + 2 * TC_BM - 1) / (2 * TC_BM), n_tiles = (n + tile_cols - 1) / tile_cols;
     const int tiles = m_pairs * n_tiles;
