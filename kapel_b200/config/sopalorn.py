@@ -163,7 +163,7 @@ def _read_mixer(kind: str, m: dict, where: str):
     mask = _record(left, "mask", f"{w}left.")
     window = SopalornWindow(*_sizes(left, f"{w}left."), _float(_flat(left, f"{w}left."), [f"{w}left.scale"], required=True, positive=False),
                             _int(_flat(mask, f"{w}left.mask."), [f"{w}left.mask.size"], hi=1 << 30))
-    delta = SopalornDelta(*_sizes(right, f"{w}right."), _int(_flat(right, f"{w}right."), [f"{w}right.conv"], hi=8))
+    delta = SopalornDelta(*_sizes(right, f"{w}right."), _int(_flat(right, f"{w}right."), [f"{w}right.conv"], hi=16))
     return SopalornParallel(window, delta)
 
 

@@ -28,7 +28,7 @@ namespace kb {
 typedef __nv_bfloat16 bf16;
 
 constexpr int DC = 4;                  // value components (warps) a block of the scan
-constexpr int DELTA_MAX_TAPS = 8;
+constexpr int DELTA_MAX_TAPS = 16;
 constexpr int DELTA_R = 8;             // memory rows a lane can hold: d <= 32 * DELTA_R
 
 struct DeltaParams {

@@ -40,8 +40,8 @@ class Delta(Part):
             raise ValueError(f"delta: {spec.num_heads} heads over {spec.num_kv_heads} key heads")
         if spec.head_dim > 256:
             raise ValueError(f"delta: a key size of {spec.head_dim} is more than the scan kernel's 256")
-        if not 1 <= spec.conv <= 8:
-            raise ValueError(f"delta: a convolution over {spec.conv} rows (1 to 8)")
+        if not 1 <= spec.conv <= 16:
+            raise ValueError(f"delta: a convolution over {spec.conv} rows (1 to 16)")
 
     def input_names(self):
         """The weights whose rows make up the stacked product, in order."""
