@@ -1,0 +1,798 @@
+"""Sopalorn on the GPU: each mechanism's kernels against the plain functions of `plain_sopalorn`, and the
+engine (step function, cache, scheduler, entry point) against the plain forward pass, on small
+configurations that differ in every size, constant and in the order of their layers."""
+import json
+
+import numpy as np
+import pytest
+import torch
+
+import plain_sopalorn as PS
+from helpers import TraceBuilder, random_tokens, rel_err, run_trace_engine
+
+pytestmark = pytest.mark.gpu
+
+
+def dense(ff, limit):
+    return {"kind": "dense", "ff": ff, "limit": limit}
+
+
+def moe(experts, identity, top, scale, ff):
+    return {"kind": "moe", "router": {"experts": experts, "identity": identity, "top": top, "scale": scale}, "expert": {"ff": ff}}
+
+
+def rotation(base, dims, scaling=None):
+    rot = {"base": base, "dims": dims}
+    if scaling is not None:
+        rot["scaling"] = dict(zip(("factor", "original", "fast", "slow"), scaling))
+    return rot
+
+
+def attention_layer(heads, kv_heads, dim, vdim, scale, rot, mlp, kv_from=None):
+    m = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "scale": scale, "rot": rot}
+    if kv_from is not None:
+        m["kv_from"] = kv_from
+    return {"type": "attention", "mixer": m, "mlp": mlp}
+
+
+def lightning_layer(dim, vdim, decay, mlp):
+    return {"type": "lightning", "mixer": {"heads": len(decay), "dim": dim, "vdim": vdim, "decay": decay}, "mlp": mlp}
+
+
+def parallel_layer(left, size, scale, right, conv, mlp):
+    names = ("heads", "kv_heads", "dim", "vdim")
+    return {"type": "parallel", "mlp": mlp, "mixer": {"left": {**dict(zip(names, left)), "scale": scale, "mask": {"size": size}},
+                                                      "right": {**dict(zip(names, right)), "conv": conv}}}
+
+
+def config(vocab, width, streams, eps, embed, logit, layers):
+    return {"architecture": "Sopalorn", "vocab": vocab, "width": width, "streams": streams, "norm": {"eps": eps}, "embedding": {"scale": embed},
+            "logit_scale": logit, "layers": layers}
+
+
+ROT_A = rotation(500.0, 12, (4.0, 64, 8.0, 1.0))
+# A: three streams, values of another size than keys (the row-wise attention), a layer that reads another's keys with more query
+# heads than that one has, identity experts, four delta heads over two key heads.
+# B: one stream, one head everywhere, filters of one weight, no scaling, no identity experts, one expert a token, layers without
+# feed-forwards, scales of 1.
+# C: keys and values of one size (the tensor-core attention in bfloat16), five streams, a window of 70, heads of 80 and 64.
+CONFIGS = {
+    "A": (config(131, 64, 3, 1e-5, 3.0, 0.5, [
+        parallel_layer((6, 2, 16, 24), 21, 0.3, (4, 2, 24, 16), 3, moe(7, 2, 3, 1.7, 40)),
+        attention_layer(6, 3, 16, 24, 0.25, ROT_A, dense(88, 0.8)),
+        lightning_layer(24, 8, [0.9375, 0.5, 0.99609375], None),
+        attention_layer(9, 3, 16, 24, 0.25, ROT_A, moe(5, 3, 2, 0.6, 24), kv_from=1),
+    ]), 51),
+    "B": (config(89, 48, 1, 1e-6, 1.0, 1.0, [
+        lightning_layer(40, 16, [0.984375], dense(56, 7.0)),
+        parallel_layer((1, 1, 32, 8), 5, 0.2, (1, 1, 16, 40), 1, None),
+        attention_layer(1, 1, 32, 32, 0.2, rotation(10000.0, 32), moe(4, 0, 1, 1.0, 32)),
+        attention_layer(1, 1, 32, 32, 0.3, rotation(10000.0, 32), None, kv_from=2),
+    ]), 52),
+    "C": (config(64, 32, 5, 1e-5, 6.0, 3.0, [
+        attention_layer(8, 2, 64, 64, 0.125, rotation(1000.0, 48, (2.0, 100, 16.0, 1.0)), dense(40, 1.5)),
+        parallel_layer((9, 3, 80, 80), 70, 0.11, (3, 3, 40, 16), 5, dense(24, 0.5)),
+        attention_layer(4, 2, 64, 64, 0.2, rotation(1000.0, 48, (2.0, 100, 16.0, 1.0)), moe(6, 1, 2, 2.5, 48), kv_from=0),
+        lightning_layer(16, 32, [0.75, 0.998046875], moe(3, 6, 4, 1.0, 16)),
+    ]), 53),
+}
+# Largest difference of logits over the largest plain logit, row by row. The 32-bit runs see a few 1e-6 and every row is held to
+# 1e-4. In bfloat16 (products and caches in bfloat16 under 32-bit norms, scores, streams and recurrences) a row is held to 3e-1, the
+# median row to 3e-2, and at most one row in twenty may be over 1e-1: a wrong key, a lost state or a forgotten sink moves every row
+# by tenths; a token whose experts are a close call may differ.
+TOL = {"float32": 1e-4, "bfloat16": 3e-1}
+
+
+def check_rows(results, builder, plain_by_request, dtype, what=""):
+    errs = []
+    for step, rows in builder.rows.items():
+        assert step in results, f"{what}: step {step} wrote no logits"
+        got = results[step]
+        assert got.shape[0] == len(rows), f"{what}: step {step}: {got.shape[0]} rows for {len(rows)} wanted"
+        for i, (rid, pos) in enumerate(rows):
+            err = rel_err(got[i], plain_by_request[rid][pos])
+            assert err <= TOL[dtype], f"{what}: step {step}, request {rid}, position {pos}: relative error {err:.3e} > {TOL[dtype]:.1e}"
+            errs.append(err)
+    errs = np.asarray(errs)
+    if dtype == "bfloat16":
+        assert np.median(errs) < 3e-2 and (errs > 1e-1).sum() <= max(1, len(errs) // 20), f"{what}: median {np.median(errs):.2e}, {(errs > 1e-1).sum()} of {len(errs)} rows over 1e-1"
+    return float(errs.max())
+
+
+def make_folder(raw, seed, tmp):
+    """A folder with random weights. Streams keep most of themselves from one sublayer to the next (as trained ones would), the window's
+    scores are sharp enough for one key to count, and routers are decided."""
+    from kapel_b200.config import config_from_json
+    from kapel_b200.weights import write_safetensors
+    from kapel_b200.weights.random_init import random_tensors
+
+    c = config_from_json(raw)
+    out = {}
+    for name, x in random_tensors(c, seed).items():
+        y = x.float()
+        if name.endswith(".mix"):
+            y = 0.3 * y + 0.8 * torch.eye(y.shape[0])
+        elif name.endswith((".in", "norm1", "norm2", "final.norm")):
+            y = y + 0.6
+        elif name.endswith(("left.q", "mlp.router")):
+            y = 3.0 * y
+        out[name] = y.to(torch.bfloat16)
+    tmp.mkdir(parents=True, exist_ok=True)
+    (tmp / "config.json").write_text(json.dumps(c.to_json()))
+    write_safetensors(tmp / "model.safetensors", out)
+    return tmp
+
+
+def read_tensors(folder):
+    """{name: float64 array} of a folder's model.safetensors, read with this file's own few lines."""
+    blob = (folder / "model.safetensors").read_bytes()
+    n = int.from_bytes(blob[:8], "little")
+    header = json.loads(blob[8 : 8 + n])
+    out = {}
+    for name, rec in header.items():
+        if name == "__metadata__":
+            continue
+        a, b = rec["data_offsets"]
+        raw = (np.frombuffer(blob[8 + n + a : 8 + n + b], dtype="<u2").astype(np.uint32) << 16).view(np.float32)
+        out[name] = raw.reshape(rec["shape"]).astype(np.float64)
+    return out
+
+
+@pytest.fixture(scope="module")
+def models(tmp_path_factory):
+    out = {}
+    for name, (raw, seed) in CONFIGS.items():
+        folder = make_folder(raw, seed, tmp_path_factory.mktemp(f"sopalorn_{name}"))
+        out[name] = (folder, raw, read_tensors(folder))
+    return out
+
+
+_PLAIN = {}
+
+
+def plain(models, name, tokens):
+    key = (name, tuple(tokens))
+    if key not in _PLAIN:
+        _, raw, t = models[name]
+        _PLAIN[key] = PS.forward(raw, t, list(tokens))
+    return _PLAIN[key]
+
+
+def dev(a, dtype=torch.float32):
+    return torch.tensor(np.asarray(a), dtype=dtype, device="cuda").contiguous()
+
+
+def bf16_round(a):
+    return torch.tensor(np.asarray(a), dtype=torch.bfloat16).double().numpy()
+
+
+def split_sum(rows):
+    """A tensor as three split-K partial sums that add up to it exactly."""
+    from kapel_b200 import kernels as K
+
+    upper = (rows.view(torch.int32) & -4096).view(torch.float32)
+    return K.SplitSum(torch.stack([upper, rows - upper, torch.zeros_like(rows)]).contiguous())
+
+
+def batch_of(step):
+    """(entry of every row, ranges, slots) on the device for a step [(name, slot, a, b)]."""
+    from kapel_b200 import kernels as K
+
+    entry = dev(np.concatenate([np.full(b - a, i) for i, (_, _, a, b) in enumerate(step)]), torch.int32)
+    return entry, K.entry_ranges(entry, len(step)), dev([s for _, s, _, _ in step], torch.int32)
+
+
+# -------------------------------------------------------------------------------------- streams
+@pytest.mark.parametrize("rows", [3, 70])
+@pytest.mark.parametrize("S,width", [(1, 48), (2, 50), (3, 64), (4, 2052), (5, 33), (8, 320), (11, 76), (16, 20)])
+def test_streams_written_and_read_in_one_kernel(S, width, rows):
+    """A branch as a tensor, as partial sums and as two normed branches; with and without a weight a channel; with a layer norm with
+    a bias, without one, and an RMS norm; write alone and read alone."""
+    from kapel_b200 import kernels as K
+
+    rng = np.random.default_rng(S * width)
+    x, y, z = rng.standard_normal((S, rows, width)) + 2.0, rng.standard_normal((rows, width)), rng.standard_normal((rows, width)) * 3
+    mix, out, w_in = rng.standard_normal((S, S)), rng.standard_normal(S), rng.standard_normal(S)
+    scale, w, b, wa, wb = (rng.standard_normal(width) for _ in range(5))
+    side = lambda a: dev(np.ascontiguousarray(np.moveaxis(a, 0, 1)).reshape(rows, S * width))
+    back = lambda t: np.moveaxis(t.double().cpu().numpy().reshape(rows, S, width), 1, 0)
+    ln = lambda u: PS.layer_norm(u, w, b, 1e-5)
+    normed = PS.rms_unit(y, 1e-4) * wa + PS.rms_unit(z, 1e-4) * wb
+    branches = {"tensor": (dev(y), y), "partial sums": (split_sum(dev(y)), y), "bfloat16": (dev(y, torch.bfloat16), bf16_round(y)),
+                "normed": (K.NormedSum(dev(y), dev(wa), dev(z), dev(wb), 1e-4), normed),
+                "normed partial sums": (K.NormedSum(split_sum(dev(y)), dev(wa), split_sum(dev(z)), dev(wb), 1e-4), normed)}
+    for what, (branch, value) in branches.items():
+        for sc in (None, scale):
+            want = PS.write_streams(x, mix, out, value if sc is None else value * sc)
+            t = side(x)
+            h = K.stream_step(t, S, (branch, None if sc is None else dev(sc), dev(mix), dev(out)), (dev(w_in), dev(w), dev(b), 1e-5, 0.0, True), torch.float32)
+            assert rel_err(back(t), want) < 3e-6, what
+            assert rel_err(h.cpu().numpy(), ln(PS.read_streams(want, w_in))) < 2e-5, what
+    t = side(x)
+    assert K.stream_step(t, S, (dev(y), None, dev(mix), dev(out))) is None
+    want = PS.write_streams(x, mix, out, y)
+    assert rel_err(back(t), want) < 3e-6
+    before = t.clone()
+    u = PS.read_streams(want, w_in)
+    reads = {"bias": ((dev(w_in), dev(w), dev(b), 1e-5, 0.0, True), ln(u)), "offset": ((dev(w_in), dev(w), None, 1e-5, 1.0, True), PS.layer_norm(u, w + 1, 0.0, 1e-5)),
+             "rms": ((dev(w_in), dev(w), None, 1e-5, 0.0, False), PS.rms_unit(u, 1e-5) * w)}
+    for what, (read, value) in reads.items():
+        for dtype, tol in ((torch.float32, 2e-5), (torch.bfloat16, 1e-2)):
+            assert rel_err(K.stream_step(t, S, None, read, dtype).float().cpu().numpy(), value) < tol, what
+    assert torch.equal(before, t)
+    pick = [rows - 1, 0, 1]
+    assert rel_err(K.stream_sum(t, S, dev(pick, torch.int32)).cpu().numpy(), want.sum(0)[pick]) < 3e-6
+
+
+def test_what_two_normed_branches_are_to_any_other_reader():
+    from kapel_b200 import kernels as K
+
+    rng = np.random.default_rng(6)
+    y, z, wa, wb = rng.standard_normal((5, 40)), rng.standard_normal((5, 40)) * 9, rng.standard_normal(40), rng.standard_normal(40)
+    want = PS.rms_unit(y, 1e-3) * wa + PS.rms_unit(z, 1e-3) * wb
+    both = K.NormedSum(split_sum(dev(y)), dev(wa), dev(z), dev(wb), 1e-3)
+    assert rel_err(K.finish(both, torch.float32).cpu().numpy(), want) < 1e-5
+    x = rng.standard_normal((5, 40))
+    t = dev(x)
+    K.add_rmsnorm(t, both, None, None, torch.float32)
+    assert rel_err(t.cpu().numpy(), x + want) < 1e-5
+
+
+@pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
+def test_embedding_rows_in_every_stream_and_layer_norm_with_a_bias(dtype):
+    from kapel_b200 import kernels as K
+
+    rng = np.random.default_rng(3)
+    table, ids = bf16_round(rng.standard_normal((20, 36))), [3, 19, 0, 3]
+    got = K.embed(dev(table, dtype), dev(ids, torch.int32), 2.5, copies=3).cpu().numpy()
+    assert np.array_equal(got, np.tile((table[ids] * 2.5).astype(np.float32), (1, 3)))
+    x, w, b = rng.standard_normal((6, 50)) + 5, bf16_round(rng.standard_normal(50)), bf16_round(rng.standard_normal(50))
+    got = K.layernorm(dev(x), dev(w, dtype), 1e-5, 0.0, torch.float32, bias=dev(b, dtype)).cpu().numpy()
+    assert rel_err(got, PS.layer_norm(x, w, b, 1e-5)) < 1e-5
+
+
+# -------------------------------------------------------------------------------------- attention
+def paged(rng, n_tokens, page_size=16, spare=3):
+    n_pages = -(-n_tokens // page_size)
+    pages = rng.permutation(n_pages + spare)[:n_pages]
+    lines = np.array([pages[p // page_size] * page_size + p % page_size for p in range(n_tokens)])
+    return n_pages + spare, pages, lines
+
+
+def plain_heads(q, k, v, scale, sinks, rows, window):
+    H, per = q.shape[1], q.shape[1] // k.shape[1]
+    out = np.zeros((len(rows), H, v.shape[2]))
+    for i, r in enumerate(rows):
+        first = max(0, r - window + 1) if window else 0
+        for h in range(H):
+            s = k[first : r + 1, h // per] @ q[i, h] * scale
+            top = max(s.max(), sinks[h])
+            p = np.exp(s - top)
+            out[i, h] = (p / (p.sum() + np.exp(sinks[h] - top))) @ v[first : r + 1, h // per]
+    return out
+
+
+class Paged:
+    """Keys and values of one request in shuffled pages, and the kernels' ways to attend to them within a window."""
+
+    def __init__(self, rng, k, v, dtype):
+        self.n_pages, pages, lines = paged(rng, len(k))
+        G, d, e = k.shape[1], k.shape[2], v.shape[2]
+        self.kt = torch.zeros((self.n_pages, G, 16, d), dtype=dtype, device="cuda")
+        self.vt = torch.zeros((self.n_pages, G, 16, e), dtype=dtype, device="cuda")
+        where = torch.tensor(lines, device="cuda")
+        self.kt[where // 16, :, where % 16] = dev(k, dtype)
+        self.vt[where // 16, :, where % 16] = dev(v, dtype)
+        self.bt = dev(np.concatenate([pages, [-1]])[None, :], torch.int32)
+        self.dtype, self.G = dtype, G
+
+    def rows(self, q, rows, scale, sinks, window):
+        from kapel_b200 import kernels as K
+
+        counts = dev(np.array(rows) + 1, torch.int32)
+        entry = torch.zeros(len(rows), dtype=torch.int32, device="cuda")
+        slots = max(rows) // K.attention_chunk() + 1
+        return K.paged_attention_rows(dev(q, self.dtype), self.kt, self.vt, self.bt, entry, counts, 16, window, scale, None, slots,
+                                      sinks=dev(sinks)).float().cpu().numpy()
+
+    def tiles(self, q, rows, scale, sinks, window, split=0):
+        """A run of rows as one portion of a prompt, the keys whole or in slots of `split`."""
+        from kapel_b200 import kernels as K
+        from kapel_b200.engine.batch import cut_tiles
+
+        assert rows == list(range(rows[0], rows[-1] + 1))
+        counts = dev(np.array(rows) + 1, torch.int32)
+        cut = tuple(dev(t, torch.int32) for t in cut_tiles(np.array([0]), np.array([len(rows)]), K.attention_mma_rows(False) // (q.shape[1] // self.G)))
+        slots = rows[-1] // split + 1 if split else 1
+        return K.paged_attention_mma(dev(q, self.dtype), self.kt, self.vt, self.bt, counts, cut, 16, window, scale, None, 0, split if slots > 1 else 0,
+                                     slots, False, sinks=dev(sinks)).float().cpu().numpy()
+
+    def decode(self, q, rows, scale, sinks, window, split=0):
+        """Every row a request of its own that brings one token (all share the pages); slots counted from the window's start."""
+        from kapel_b200 import kernels as K
+
+        n, per = len(rows), q.shape[1] // self.G
+        counts = dev(np.array(rows) + 1, torch.int32)
+        tiles = (dev(np.arange(n), torch.int32), dev(np.arange(n), torch.int32), dev(np.ones(n), torch.int32))
+        span = min(max(rows) + 1, window) if window else max(rows) + 1
+        slots = -(-span // split) if split else 1
+        return K.paged_attention_mma(dev(q, self.dtype), self.kt, self.vt, self.bt.repeat(n, 1).contiguous(), counts, tiles, 16, window, scale, None, per,
+                                     split, slots, True, sinks=dev(sinks)).float().cpu().numpy()
+
+
+WAYS = ["rows f32", "rows bf16", "prompt", "prompt in slots", "decode", "decode in slots"]
+
+
+def attend(way, cache, q, rows, scale, sinks, window):
+    if way.startswith("rows"):
+        return np.concatenate([cache.rows(q[i : i + 1], [r], scale, sinks, window) for i, r in enumerate(rows)])
+    if way == "prompt":
+        return cache.tiles(q, rows, scale, sinks, window)
+    if way == "prompt in slots":
+        return cache.tiles(q, rows, scale, sinks, window, split=128)
+    split = 64 if way == "decode in slots" else 0
+    return np.concatenate([cache.decode(q[i : i + 8], rows[i : i + 8], scale, sinks, window, split) for i in range(0, len(rows), 8)])
+
+
+@pytest.mark.parametrize("way", WAYS)
+@pytest.mark.parametrize("H,G,d,window", [(9, 3, 80, 70), (10, 2, 64, 1), (4, 4, 128, 300), (16, 1, 32, 64), (6, 2, 96, 17), (3, 1, 48, 2000), (6, 3, 96, None)])
+def test_attention_with_a_sink_within_a_window_on_every_kernel(way, H, G, d, window):
+    rng = np.random.default_rng(H * d)
+    dtype = torch.float32 if way == "rows f32" else torch.bfloat16
+    T = 500
+    k, v = rng.standard_normal((T, G, d)), rng.standard_normal((T, G, d))
+    rows = list(range(390, 500)) if way.startswith("prompt") else [0, 1, 15, 16, 63, 64, 69, 70, 71, 255, 256, 300, 499]
+    q = rng.standard_normal((len(rows), H, d))
+    if dtype == torch.bfloat16:
+        q, k, v = bf16_round(q), bf16_round(k), bf16_round(v)
+    cache = Paged(rng, k, v, dtype)
+    for sinks in (rng.standard_normal(H) * 2, np.zeros(H), np.full(H, 9.0)):
+        want = plain_heads(q, k, v, 0.2, sinks, rows, window)
+        assert rel_err(attend(way, cache, q, rows, 0.2, sinks, window), want) < (1e-5 if dtype == torch.float32 else 2e-2), sinks
+    if way.startswith("prompt"):                             # the first tokens of a sequence
+        rows = list(range(90))
+        q = bf16_round(rng.standard_normal((90, H, d)))
+        assert rel_err(attend(way, cache, q, rows, 0.2, np.full(H, 0.5), window), plain_heads(q, k, v, 0.2, np.full(H, 0.5), rows, window)) < 2e-2
+
+
+@pytest.mark.parametrize("way", WAYS)
+def test_a_windows_edge_and_a_sink_that_show(way):
+    """One key stands out by 20 against a query. Rows that have it just inside their window see it alone (a sink as high halves it), rows
+    that have it just outside do not see it at all, wherever it lies: at the start, at page and tile borders."""
+    rng = np.random.default_rng(3)
+    dtype, tol = (torch.float32, 1e-4) if way == "rows f32" else (torch.bfloat16, 3e-2)
+    H, d, T, window = 2, 64, 420, 77
+    for target in (0, 1, 15, 16, 63, 64, 127, 128, 200, 255, 256, 300):
+        k, v = bf16_round(rng.standard_normal((T, 1, d)) * 0.2), bf16_round(rng.standard_normal((T, 1, d)))
+        k[:, 0, 0] = 0.0
+        k[target, 0] = 0.0
+        k[target, 0, 0] = 1.0
+        last = target + window - 1                           # the last row that sees it
+        rows = list(range(last - 9, last + 11)) if way.startswith("prompt") else [target, last - 1, last, last + 1, last + 2]
+        q = bf16_round(rng.standard_normal((len(rows), H, d)) * 0.1)
+        q[..., 0] = 20.0
+        cache = Paged(rng, k, v, dtype)
+        y = attend(way, cache, q, rows, 1.0, np.array([-30.0, 20.0]), window)
+        inside = np.array([r <= last for r in rows])
+        assert np.abs(y[inside, 0] - v[target, 0]).max() < tol * 3, target
+        assert np.abs(y[inside, 1] - 0.5 * v[target, 0]).max() < tol * 3, target
+        assert np.abs(y[~inside, 1]).max() < 1e-5, target    # without the key the sink takes everything
+        want = plain_heads(q, k, v, 1.0, np.array([-30.0, 20.0]), rows, window)
+        assert rel_err(y, want) < tol, target
+
+
+@pytest.mark.parametrize("dtype,tol", [(torch.float32, 1e-5), (torch.bfloat16, 1e-2)])
+@pytest.mark.parametrize("H,d,rotary", [(6, 16, 12), (1, 40, 40), (5, 96, 24), (3, 10, 2)])
+def test_queries_alone_normed_and_turned(H, d, rotary, dtype, tol):
+    """What a layer does that reads another layer's keys: nothing of the cache is touched."""
+    from kapel_b200 import kernels as K
+
+    rng = np.random.default_rng(H * d)
+    rows = 7
+    x, w = rng.standard_normal((rows, 3 + H * d)), bf16_round(rng.standard_normal(H * d))
+    positions = np.array([0, 1, 2, 63, 64, 1000, 5])
+    rot = rotation(300.0, rotary, (3.0, 80, 8.0, 1.0))
+    f, m = PS.frequencies(rot)
+    table = K.rope_table_freqs(dev(positions, torch.int32), dev(f, torch.float64), m)
+    want = PS.rotate_neighbours((PS.rms_unit(x[:, 3:], 1e-4) * w).reshape(rows, H, d), positions, rot)
+    for src in (dev(x), split_sum(dev(x))):
+        q, kept = K.proj_rope_append(src, 3, 3 + H * d, 3 + H * d, None, (dev(w, dtype), 1e-4, 0.0), None, table, rotary, True, None, None, False, None, None,
+                                     None, H, 0, d, d, False, dtype)
+        assert kept is None and rel_err(q.float().cpu().numpy(), want) < tol
+
+
+# -------------------------------------------------------------------------------------- memories, gates, experts
+LENGTHS = {"a": 300, "b": 37, "c": 40}
+
+
+def walk(run, states):
+    """Three requests of unequal length; whole; then in portions down to two tokens beside each other's single tokens; a request
+    that ends and whose slot the next one takes."""
+    run([("a", 1, 0, 300), ("b", 2, 0, 37)])
+    for s in states:
+        s.zero_()
+    run([("a", 1, 0, 2), ("b", 2, 0, 30)])
+    run([("b", 2, 30, 31), ("a", 1, 2, 99)])
+    for i in range(6):
+        run([("a", 1, 99 + 2 * i, 101 + 2 * i), ("b", 2, 31 + i, 32 + i)])
+    for s in states:
+        s[2].zero_()                                         # b is finished; c takes its slot
+    run([("c", 2, 0, 3), ("a", 1, 111, 300)])
+    for i in range(3, 40):
+        run([("c", 2, i, i + 1)])
+
+
+def rows_of(data, step):
+    rows = dev(np.concatenate([data[m][a:b] for m, _, a, b in step]))
+    return split_sum(rows) if len(rows) <= 4 else rows
+
+
+def compare(out, want, step, tol):
+    at = 0
+    for m, _, a, b in step:
+        err = float(np.abs(out[at : at + b - a] - want[m][a:b]).max() / np.abs(want[m]).max())
+        assert err < tol, f"{m}[{a}:{b}]: {err:.2e}"
+        at += b - a
+
+
+@pytest.fixture
+def chunk_rows(request):
+    from kapel_b200 import kernels as K
+
+    K.retention_chunk_rows(request.param)
+    yield request.param
+    K.retention_chunk_rows(-1)
+
+
+@pytest.mark.parametrize("chunk_rows", [0, 1, -1], indirect=True)        # row by row; by chunks whatever a portion's length; the launcher's choice
+@pytest.mark.parametrize("H,d,e", [(3, 24, 8), (1, 40, 16), (2, 64, 64), (2, 130, 5)])
+def test_decaying_memory_behind_silu_in_portions_and_token_by_token(H, d, e, chunk_rows):
+    from kapel_b200 import kernels as K
+
+    rng = np.random.default_rng(d + e)
+    nq, nv = H * d, H * e
+    decay = [0.998046875, 0.60625, 1.0][:H]
+    data, want = {}, {}
+    for name, T in LENGTHS.items():
+        x = data[name] = rng.standard_normal((T, 3 + 2 * nq + nv))
+        y = PS.silu(x[:, 3:])
+        q, k, v = y[:, :nq].reshape(T, H, d), y[:, nq : 2 * nq].reshape(T, H, d), y[:, 2 * nq :].reshape(T, H, e)
+        want[name] = np.stack([PS.decay_recurrence(q[:, h], k[:, h], v[:, h], decay[h]) for h in range(H)], axis=1)
+    state = torch.zeros((3, nq * e), dtype=torch.float32, device="cuda")
+
+    def run(step):
+        entry, ranges, slots = batch_of(step)
+        out = K.retention_scan(rows_of(data, step), 3, 3 + nq, 3 + 2 * nq, dev(decay), None, 0, 1.0, state, ranges, slots, len(step),
+                               max(b - a for _, _, a, b in step), H, d, e, act="silu").cpu().numpy()
+        compare(out, want, step, 5e-5)
+
+    walk(run, [state])
+
+
+def test_delta_rule_with_long_filters_in_the_columns_of_a_wider_product():
+    from kapel_b200 import kernels as K
+
+    rng = np.random.default_rng(9)
+    H, G, d, e, taps, off = 4, 2, 24, 16, 13, 7
+    n, nv = G * d, H * e
+    conv, alog, dt = rng.standard_normal((2 * n + nv, taps)) * 0.4, rng.standard_normal(H), rng.standard_normal(H)
+    b_off = off + 2 * n + 2 * nv
+    data, want = {}, {}
+    for name, T in LENGTHS.items():
+        x = data[name] = rng.standard_normal((T, b_off + 2 * H))
+        c = PS.silu(PS.short_conv(x[:, off : off + 2 * n + nv], conv))
+        q, k = PS.unit_vectors(c[:, :n].reshape(T, G, d)) * d ** -0.5, PS.unit_vectors(c[:, n : 2 * n].reshape(T, G, d))
+        v = c[:, 2 * n :].reshape(T, H, e)
+        beta, g = PS.sigmoid(x[:, b_off : b_off + H]), np.exp(-np.exp(alog) * PS.softplus(x[:, b_off + H :] + dt))
+        want[name] = np.stack([PS.delta_recurrence(q[:, h // 2], k[:, h // 2], v[:, h], g[:, h], beta[:, h]) for h in range(H)], axis=1)
+    state = torch.zeros((3, K.delta_state_floats(H, G, d, e, taps)), dtype=torch.float32, device="cuda")
+
+    def run(step):
+        entry, ranges, slots = batch_of(step)
+        out = K.delta_scan(rows_of(data, step), off, off + n, off + 2 * n, b_off, b_off + H, dev(conv), dev(alog), dev(dt), state, entry, ranges, slots,
+                           len(step), H, G, d, e, taps, d ** -0.5, 1e-6).cpu().numpy()
+        compare(out, want, step, 5e-5)
+
+    walk(run, [state])
+
+
+@pytest.mark.parametrize("rows", [2, 65])
+@pytest.mark.parametrize("width", [24, 511, 512, 1536])
+def test_a_whole_row_normed_and_gated(width, rows):
+    from kapel_b200 import kernels as K
+
+    rng = np.random.default_rng(width)
+    y, z, w = rng.standard_normal((rows, width)), rng.standard_normal((rows, 2 + width)), rng.standard_normal(width)
+    want = PS.rms_unit(y, 1e-4) * w * PS.sigmoid(z[:, 2:])
+    for gate in (dev(z), split_sum(dev(z))):
+        got = K.head_gate(dev(y).view(rows, 1, width), gate, 2, dev(w), True, 1e-4, torch.float32, pad_to=width + 5).cpu().numpy()
+        assert rel_err(got[:, :width], want) < 1e-5 and (got[:, width:] == 0).all()
+    two = K.head_gate(dev(np.stack([y, 2 * y], 1)), dev(np.concatenate([z, z[:, 2:]], 1)), 2, dev(np.concatenate([w, w])), False, 0.0, torch.float32,
+                      gate_act="silu").cpu().numpy()
+    assert rel_err(two, np.concatenate([y * w * PS.silu(z[:, 2:]), 2 * y * w * PS.silu(z[:, 2:])], 1)) < 1e-5
+
+
+@pytest.mark.parametrize("experts,identity,top,scale", [(7, 2, 3, 1.7), (4, 0, 1, 1.0), (3, 6, 4, 0.4), (1, 1, 2, 2.0)])
+def test_router_with_identity_experts_and_a_scale(experts, identity, top, scale):
+    from kapel_b200 import kernels as K
+
+    rng = np.random.default_rng(experts)
+    rows, width, n = 90, 40, experts + identity
+    h, router, correction = rng.standard_normal((rows, width)), rng.standard_normal((n, width)), rng.standard_normal(n) * 0.2
+    got_e, got_w = (t.cpu().numpy() for t in K.moe_route(dev(h), dev(router), dev(correction), top, 1, 1, 2, "softmax", True, scale))
+    want = np.zeros((rows, width))
+    y = rng.standard_normal((rows * top, width))
+    for r in range(rows):
+        e, w = PS.route(router @ h[r], correction, top, scale)
+        assert list(got_e[r]) == list(e) and np.allclose(got_w[r], w, rtol=2e-5)
+        for t in range(top):
+            want[r] += w[t] * (y[r * top + t] if e[t] < experts else h[r])
+    lists = K.moe_sort(dev(got_e, torch.int32), experts)
+    assert int(lists.offsets[experts]) == int((got_e < experts).sum())            # identity pairs are in no list
+    ys = dev(y)
+    ys[torch.tensor(got_e.reshape(-1) >= experts, device="cuda")] = float("nan")  # nobody writes their rows, nobody reads them
+    got = K.moe_combine(ys, dev(got_w), torch.float32, experts=dev(got_e, torch.int32), real=experts, own=dev(h)).cpu().numpy()
+    assert rel_err(got, want) < 1e-5
+    got = K.moe_combine(ys, dev(got_w), torch.float32, experts=dev(got_e, torch.int32), real=experts, own=dev(h, torch.bfloat16)).cpu().numpy()
+    assert rel_err(got, want) < 1e-2
+
+
+@pytest.mark.parametrize("rows", [1, 5, 17, 40, 64, 65, 200, 300])
+@pytest.mark.parametrize("n,k", [(40, 64), (384, 320), (1000, 128)])
+def test_bounded_unit_in_the_products_epilogue(rows, n, k):
+    from kapel_b200 import kernels as K
+
+    rng = np.random.default_rng(n + rows)
+    h, gate, up = (bf16_round(rng.standard_normal(s)) for s in ((rows, k), (n, k), (n, k)))
+    g, u = np.minimum(h @ gate.T, 3.0), np.clip(h @ up.T, -3.0, 3.0)
+    want = g * PS.sigmoid(1.702 * g) * (u + 1.0)
+    got = K.gemm_glu_fused(dev(h, torch.bfloat16), dev(np.concatenate([gate, up]), torch.bfloat16), "clamped_swish", 3.0, 1.702)
+    assert got is not None and rel_err(got.float().cpu().numpy(), want) < 1e-2
+    assert np.abs(got.float().cpu().numpy() - want).mean() < 2e-3 * np.abs(want).max()
+
+
+# -------------------------------------------------------------------------------------- the engine
+def engine_for(models, name, dtype, **kw):
+    from kapel_b200.engine import Engine
+
+    kw.setdefault("max_tokens", 1024)
+    kw.setdefault("max_sequences", 4)
+    return Engine.from_dir(models[name][0], dtype=dtype, **kw)
+
+
+def test_whose_keys_a_layer_reads_and_the_shared_product(models):
+    eng = engine_for(models, "A", "float32")
+    assert sorted(str(k) for k in eng.cache.states) == sorted(str(k) for k in ((0, "right"), 2))
+    mixer, borrowing = eng.model.blocks[0].mixer, eng.model.blocks[3].mixer
+    assert mixer.w_in.shape == (6 * 16 + 2 * 16 + 2 * 24 + 2 * 2 * 24 + 2 * 4 * 16 + 2 * 4, 64)       # one product for both sides
+    assert mixer.w_left.shape == (64, 6 * 24) and mixer.w_right.shape == (64, 4 * 16)
+    assert borrowing.w_qkv.shape == (9 * 16, 64) and eng.spec.schedule[3].cache_of == 1
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+@pytest.mark.parametrize("name", ["A", "B", "C"])
+def test_whole_prompts_portions_and_decoding_against_plain(models, name, dtype):
+    """A prompt whole; the same prompt in portions of changing size down to two tokens and then token by token (a long decoding that
+    crosses pages and windows); logits at every position."""
+    raw = models[name][1]
+    tokens = random_tokens(np.random.default_rng(7), 220, raw["vocab"])
+    want = {"w": plain(models, name, tokens), "p": plain(models, name, tokens)}
+    eng = engine_for(models, name, dtype)
+    tb = TraceBuilder()
+    tb.step([("w", tokens, range(len(tokens)))], end=["w"])
+    at = 0
+    for n in (2, 17, 3, 2, 40, 5, 65):
+        tb.step([("p", tokens[at : at + n], range(n))])
+        at += n
+    while at < len(tokens):
+        tb.step([("p", tokens[at : at + 1], [0])], end=(["p"] if at + 1 == len(tokens) else []))
+        at += 1
+    worst = check_rows(run_trace_engine(eng, tb.steps), tb, want, dtype, f"{name} {dtype}")
+    print(f"sopalorn {name} {dtype}: worst {worst:.2e}")
+    assert eng.cache.free_pages() == eng.cache.total_pages() and eng.cache.free_slots() == 4
+
+
+@pytest.mark.parametrize("name", ["A", "B", "C"])
+def test_the_streams_sum_after_every_layer_against_plain(models, name):
+    from kapel_b200.engine import StepEntry
+
+    folder, raw, t = models[name]
+    tokens = random_tokens(np.random.default_rng(1), 150, raw["vocab"])
+    plain_runs = []
+    PS.forward(raw, t, tokens, plain_runs)
+    eng = engine_for(models, name, "float32")
+    seen = []
+    eng.model.tap = lambda i, x: seen.append(x.detach().view(len(tokens), raw["streams"], -1).sum(1).cpu().numpy())
+    eng.step([StepEntry("r", tokens, [])])
+    assert len(seen) == len(plain_runs) == 4
+    for i, (got, want) in enumerate(zip(seen, plain_runs)):
+        assert rel_err(got, want) < 2e-5, f"layer {i}"
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+@pytest.mark.parametrize("name", ["A", "C"])
+def test_mixed_batches_and_reused_slots_against_each_alone(models, name, dtype):
+    """Up to four unequal requests a step, portions beside single tokens, a request left out of a step, requests that end
+    and whose pages and slots the next ones take; a pool of few pages."""
+    raw = models[name][1]
+    rng = np.random.default_rng(8)
+    reqs = {k: random_tokens(rng, n, raw["vocab"]) for k, n in dict(a=250, b=41, c=23, d=70, e=33, f=18).items()}
+    want = {k: plain(models, name, v) for k, v in reqs.items()}
+    eng = engine_for(models, name, dtype, max_tokens=64 * 3 + 256 + 64)
+    tb = TraceBuilder()
+    fed = {k: 0 for k in reqs}
+
+    def take(k, n, want_all=True):
+        a = fed[k]
+        n = min(n, len(reqs[k]) - a)
+        fed[k] += n
+        return (k, reqs[k][a : a + n], list(range(n)) if want_all else [n - 1])
+
+    done = lambda k: fed[k] == len(reqs[k])
+    tb.step([take("a", 30), take("b", 2), take("c", 23)], end=["c"])
+    tb.step([take("a", 1), take("b", 20), take("d", 17)])
+    tb.step([take("b", 1), take("d", 2), take("e", 33, False)], end=["e"])            # a is left out of this step
+    tb.step([take("d", 1), take("a", 190), take("b", 1), take("f", 5)])
+    while not all(done(k) for k in "abdf"):
+        entries = [take(k, 1) for k in "abdf" if not done(k)]
+        tb.step(entries, end=[k for k, _, _ in entries if done(k)])
+    worst = check_rows(run_trace_engine(eng, tb.steps), tb, want, dtype, f"{name} {dtype}")
+    print(f"sopalorn mixed {name} {dtype}: worst {worst:.2e}")
+    eng.cache.check()
+    assert eng.cache.free_pages() == eng.cache.total_pages() and eng.cache.free_slots() == 4
+
+
+def test_recorded_passes_leave_the_state_as_eager_ones_do(models):
+    """A prompt pass of a shape seen before and a decoding pass go through recordings, whose first eager run must not
+    advance the memories or the convolutions' history a second time."""
+    raw = models["C"][1]
+    outs = []
+    for graphs in (False, True):
+        eng = engine_for(models, "C", "float32", graphs=graphs)
+        tb = TraceBuilder()
+        for k in ("x", "y", "z"):
+            tokens = random_tokens(np.random.default_rng(ord(k)), 150, raw["vocab"])
+            tb.step([(k, tokens[:140], [139])])
+            for i in range(140, 150):
+                tb.step([(k, tokens[i : i + 1], [0])], end=([k] if i == 149 else []))
+        outs.append(run_trace_engine(eng, tb.steps))
+        if graphs:
+            assert eng.recorded_passes > 0
+    for step in outs[0]:
+        assert rel_err(outs[1][step], outs[0][step]) < 2e-6, f"step {step}"
+
+
+def test_nothing_is_read_that_nobody_wrote(models):
+    """Every fresh buffer starts as NaN (rows of identity experts' pairs stay so): the logits are the same."""
+    from kapel_b200 import kernels as K
+
+    raw = models["A"][1]
+    tokens = random_tokens(np.random.default_rng(2), 90, raw["vocab"])
+    want = {"a": plain(models, "A", tokens)}
+    K.set_poison(True)
+    try:
+        for dtype in ("float32", "bfloat16"):
+            tb = TraceBuilder()
+            tb.step([("a", tokens[:80], range(80))])
+            for i in range(80, 90):
+                tb.step([("a", tokens[i : i + 1], [0])])
+            check_rows(run_trace_engine(engine_for(models, "A", dtype), tb.steps), tb, want, dtype, dtype)
+    finally:
+        K.set_poison(False)
+
+
+ODD = config(77, 52, 2, 1e-6, 2.0, 0.7, [
+    parallel_layer((3, 1, 10, 7), 13, 0.3, (3, 1, 10, 7), 3, dense(19, 0.9)),
+    attention_layer(34, 2, 16, 16, 0.25, rotation(60.0, 6, (2.0, 30, 2.0, 1.0)), moe(3, 2, 2, 1.3, 13)),
+    lightning_layer(9, 5, [0.9, 0.5, 0.99], dense(21, 2.0)),
+    attention_layer(2, 2, 16, 16, 0.25, rotation(60.0, 6, (2.0, 30, 2.0, 1.0)), None, kv_from=1)])
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+def test_sizes_that_are_no_multiples_of_eight(dtype, tmp_path):
+    """Nor anything else; and 17 query heads a kv head, more than the tensor-core attention takes, over keys that a layer of one query
+    head a kv head reads too."""
+    from kapel_b200.engine import Engine
+
+    folder = make_folder(ODD, 6, tmp_path)
+    t = read_tensors(folder)
+    eng = Engine.from_dir(folder, dtype=dtype, max_tokens=512, max_sequences=4)
+    tokens = random_tokens(np.random.default_rng(3), 165, ODD["vocab"])
+    want = {"a": PS.forward(ODD, t, tokens)}
+    tb = TraceBuilder()
+    tb.step([("a", tokens[:140], range(140))])
+    tb.step([("a", tokens[140:143], range(3))])
+    for i in range(143, 165):
+        tb.step([("a", tokens[i : i + 1], [0])], end=(["a"] if i == 164 else []))
+    check_rows(run_trace_engine(eng, tb.steps), tb, want, dtype, f"odd {dtype}")
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+def test_a_prompt_longer_than_the_attention_kernels_chunks(models, dtype):
+    """700 tokens: the kernels' key slots are merged with the one in the denominator; portions that start in the middle of a chunk; then
+    single tokens beside another request."""
+    raw = models["C"][1]
+    tokens = random_tokens(np.random.default_rng(12), 700, raw["vocab"])
+    short = random_tokens(np.random.default_rng(13), 30, raw["vocab"])
+    want = {"a": plain(models, "C", tokens), "b": plain(models, "C", short)}
+    eng = engine_for(models, "C", dtype)
+    tb = TraceBuilder()
+    tb.step([("a", tokens[:300], [0, 1, 63, 64, 69, 70, 71, 255, 256, 299])])
+    tb.step([("b", short[:20], [19]), ("a", tokens[300:690], [0, 29, 211, 212, 389])])
+    for i in range(690, 700):
+        tb.step([("a", tokens[i : i + 1], [0]), ("b", short[i - 670 : i - 669], [0])], end=(["a", "b"] if i == 699 else []))
+    check_rows(run_trace_engine(eng, tb.steps), tb, want, dtype, "long")
+
+
+def test_a_windowed_layer_gives_its_pages_back_and_the_others_keep_theirs(models):
+    """While a request decodes past its window the windowed group's pages stay few; the keys another layer reads stay all."""
+    from kapel_b200.engine import StepEntry
+
+    eng = engine_for(models, "A", "bfloat16", max_tokens=320)
+    tokens = random_tokens(np.random.default_rng(5), 300, 131)
+    eng.step([StepEntry("a", tokens[:200], [])])
+    for i in range(200, 300):
+        eng.step([StepEntry("a", tokens[i : i + 1], [0])])
+    window, whole = sorted(total - free for total, free in zip(eng.cache.total_pages(), eng.cache.free_pages()))
+    assert whole >= 300 // 16 and window <= 4
+    eng.end("a")
+    assert eng.cache.free_pages() == eng.cache.total_pages()
+
+
+@pytest.mark.parametrize("name", ["A", "B", "C"])
+def test_greedy_generation_through_the_entry_point_and_scheduler(models, name):
+    import kapel_b200
+
+    folder, raw, t = models[name]
+    rng = np.random.default_rng(10)
+    prompts = [random_tokens(rng, n, raw["vocab"]) for n in (3, 29, 75)]
+
+    def plain_greedy(prompt, n):
+        seq, margins = list(prompt), []
+        for _ in range(n):
+            row = PS.forward(raw, t, seq)[-1]
+            order = np.argsort(row)
+            margins.append(float(row[order[-1]] - row[order[-2]]))
+            seq.append(int(order[-1]))
+        return seq[len(prompt):], margins
+
+    want = [plain_greedy(p, 12) for p in prompts]
+    model = kapel_b200.Model(str(folder), dtype="f32", max_tokens_cached=1024, max_sequences=4, max_pass_tokens=32)
+    for p, (tokens, margins) in zip(prompts, want):
+        safe = next((i for i, m in enumerate(margins) if m < 1e-3), len(margins))
+        assert model.generate(p, max_tokens=12)[:safe] == tokens[:safe]
+    together = model.generate_batch(prompts, max_tokens=12)
+    for got, (tokens, margins) in zip(together, want):
+        safe = next((i for i, m in enumerate(margins) if m < 1e-3), len(margins))
+        assert got[:safe] == tokens[:safe]
+    assert model.engine.cache.free_pages() == model.engine.cache.total_pages()
+
+
+def test_replay_program_and_command_line(models, tmp_path):
+    import subprocess
+    import sys
+
+    import kapel_b200
+    from helpers import ROOT
+
+    folder, raw, _ = models["A"]
+    tokens = random_tokens(np.random.default_rng(4), 40, raw["vocab"])
+    want = plain(models, "A", tokens)
+    steps = [{"step": 0, "entries": [{"id": "q", "tokens": tokens[:33], "want": [0, 32]}], "end": []},
+             {"step": 1, "entries": [{"id": "q", "tokens": tokens[33:35], "want": []}], "end": []},
+             {"step": 5, "entries": [{"id": "q", "tokens": tokens[35:], "want": [4]}], "end": ["q"]}]
+    out = tmp_path / "logits"
+    r = subprocess.run([sys.executable, str(ROOT / "bin" / "trace_run"), "--model", str(folder), "--dtype", "float32", "--out", str(out),
+                        "--max-tokens", "64"], input="".join(json.dumps(x) + "\n" for x in steps), capture_output=True, text=True, timeout=900)
+    assert r.returncode == 0, r.stderr
+    assert [l for l in r.stdout.splitlines() if l.startswith("done ")] == ["done 0", "done 1", "done 5"]
+    first = np.fromfile(out / "0.f32", dtype="<f4").reshape(2, raw["vocab"])
+    last = np.fromfile(out / "5.f32", dtype="<f4").reshape(1, raw["vocab"])
+    assert rel_err(first, want[[0, 32]]) < TOL["float32"] and rel_err(last, want[[39]]) < TOL["float32"]
+
+    model = kapel_b200.Model(str(folder), dtype="f32", max_tokens_cached=256, max_sequences=2)
+    expect = model.generate(tokens[:9], max_tokens=6)
+    r = subprocess.run([sys.executable, "-m", "kapel_b200", "run", str(folder), "--tokens", ",".join(map(str, tokens[:9])), "--max-tokens", "6",
+                        "--greedy", "--dtype", "f32"], capture_output=True, text=True, timeout=900, cwd=str(ROOT))
+    assert r.returncode == 0, r.stderr
+    assert [int(x) for x in r.stdout.strip().splitlines()[0].split(",")] == expect
