@@ -1,7 +1,7 @@
 """Throughput of the engine at Gemma 2 sizes with random weights, on one GPU.
 
     python bench.py [--gpus 1] [--steps K] [--warmup W] [--size 2b|9b|27b] [--layers L] [--impl reference]
-    python bench.py --design fusitar|kofutar|teluzen|lokedra|mukunex [--design-sizes s,m]      (another line: see `design_line`)
+    python bench.py --design fusitar|kofutar|teluzen|lokedra|mukunex|sopalorn [--design-sizes s,m]      (another line: see `design_line`)
 
 A "step" is one decode step. The default run has the layer sizes of the 2B configuration
 (26 layers, hidden 2304, 8 heads over 4 kv heads of 256, intermediate 9216, vocabulary 256000,
@@ -473,6 +473,31 @@ def mukunex_config(z):
             "layers": [(par, lru, par, rec)[i % 4] for i in range(z["layers"])]}
 
 
+# --design sopalorn: the Sopalorn design (several residual streams; attention with norms over the whole projections and 1 in
+# the denominator, some of it over another layer's keys; windowed attention with a sink beside the gated delta rule over one
+# product, each side normed; linear attention with a fixed decay behind silu; bounded dense feed-forwards, silu-gated experts
+# some of which are the identity) beside Mukunex, the engine's other design with a fixed decay's memory and attention with a sink
+# on the same kernels, Kofutar, its other design with the gated delta rule, and Lokedra, its other design with experts on the same
+# kernels, at equal sizes: the same width, heads, head size, window, vocabulary, as many layers, dense feed-forwards and
+# experts of the same size. Its layers take turns: parallel, attention, linear attention, attention over the keys of the
+# attention layer before it; experts in the first and the last of the four.
+SOPALORN_STREAMS = 4
+
+
+def sopalorn_config(z):
+    dense = {"kind": "dense", "ff": z["top"] * z["ff"], "limit": 7.0}
+    moe = {"kind": "moe", "expert": {"ff": z["ff"]}, "router": {"experts": z["experts"], "identity": z["experts"] // 4, "top": z["top"], "scale": 1.0}}
+    heads = {"heads": z["heads"], "kv_heads": z["kv_heads"], "dim": z["dim"], "vdim": z["dim"]}
+    rot = {"base": 10000.0, "dims": z["dim"] // 2, "scaling": {"factor": 8.0, "original": 1024, "fast": 32.0, "slow": 1.0}}
+    att = lambda kv_from, mlp: {"type": "attention", "mlp": mlp, "mixer": {**heads, "scale": z["dim"] ** -0.5, "rot": rot, "kv_from": kv_from}}
+    par = {"type": "parallel", "mlp": moe, "mixer": {"left": {**heads, "scale": z["dim"] ** -0.5, "mask": {"size": z["window"]}}, "right": {**heads, "conv": 4}}}
+    lin = {"type": "lightning", "mlp": dense, "mixer": {"heads": z["heads"], "dim": z["dim"], "vdim": z["dim"],
+                                                        "decay": [1.0 - 2.0 ** -(5 + i % 8) for i in range(z["heads"])]}}
+    return {"architecture": "Sopalorn", "vocab": z["vocab"], "width": z["width"], "streams": SOPALORN_STREAMS, "norm": {"eps": 1e-6},
+            "embedding": {"scale": 1.0}, "logit_scale": 1.0,
+            "layers": [(par, att(None, dense), lin, att(i - 2, moe))[i % 4] for i in range(z["layers"])]}
+
+
 def gemma_config(z):
     return {"architectures": ["Gemma2ForCausalLM"], "model_type": "gemma2", "num_hidden_layers": z["layers"], "hidden_size": z["width"],
             "num_attention_heads": z["heads"], "num_key_value_heads": z["kv_heads"], "head_dim": z["dim"],
@@ -512,6 +537,24 @@ def design_kernel_rooflines(which, z, kind, rows, context, batch, pk):
         return {"attention": ("bytes", par_layers * batch * context * hkv * d * 2 * 2.0), "feed_forward": ("bytes", layers * 3.0 * ff * w * 2),
                 "retention_scan": ("bytes", par_layers * state), "delta_scan": ("bytes", rec_layers * state),
                 "recurrent_unit": ("bytes", lru_layers * (2.0 * w * d * 2 + batch * w * (4 + 4 + 2 + 4 * 2 * 4.0)))}
+    if which == "sopalorn":
+        par_layers, att_layers, lin_layers = (layers + 3) // 4, (layers + 2) // 4 + layers // 4, (layers + 1) // 4
+        moe_layers, dense_layers = (layers + 3) // 4 + layers // 4, (layers + 2) // 4 + (layers + 1) // 4
+        # the streams move in and out in 32-bit and the sublayer's result in, its next input out, once a sublayer (and the first input)
+        streams = ("bytes", 2 * layers * (rows if kind == "prefill" else batch) * w * (SOPALORN_STREAMS * 8 + 2 + 2.0))
+        real = z["experts"] / (z["experts"] + z["experts"] // 4)          # the share of a token's experts that are not the identity, by chance
+        if kind == "prefill":
+            pairs, seen = rows * (rows + 1) // 2, sum(min(c, win) for c in range(1, rows + 1))
+            return {"attention": ("flops", 4.0 * (att_layers * pairs + par_layers * seen) * hq * d), "sum_and_norm": streams,
+                    "feed_forward": ("flops", 2.0 * rows * 3 * z["top"] * z["ff"] * w * dense_layers),
+                    "experts": ("flops", 2.0 * rows * 3 * z["top"] * z["ff"] * w * moe_layers * real),
+                    "retention_scan": ("flops", lin_layers * 5.0 * rows * hq * d * d), "delta_scan": ("flops", par_layers * 7.0 * rows * hq * d * d)}
+        state = batch * hq * d * d * 4 * 2.0
+        experts_read = min(z["experts"], batch * z["top"] * real)
+        return {"attention": ("bytes", (att_layers * context + par_layers * min(context, win)) * batch * hkv * d * 2 * 2.0), "sum_and_norm": streams,
+                "feed_forward": ("bytes", 3.0 * z["ff"] * w * 2 * dense_layers * z["top"]),
+                "experts": ("bytes", 3.0 * z["ff"] * w * 2 * moe_layers * experts_read),
+                "retention_scan": ("bytes", lin_layers * state), "delta_scan": ("bytes", par_layers * state)}
     if which == "lokedra":
         par_layers, lat_layers, rec_layers = (layers + 3) // 4, (layers + 1) // 4, layers // 2
         r, kv = 64, KOFUTAR_KV_RANK
@@ -600,6 +643,20 @@ MUKUNEX_KERNEL_CLASSES = {
 }
 
 
+# Sopalorn's attention runs the tensor-core kernels with a sink, as Mukunex's and Kofutar's does; its dense feed-forwards the fused
+# gated products, its experts the grouped ones, as Lokedra's do; its memories are Mukunex's retention and Kofutar's delta rule. The sum of a
+# sublayer's result and the norm behind it is over several streams (`SUM_AND_NORM`: what the designs of one stream run there).
+SOPALORN_KERNEL_CLASSES = {
+    "attention": ("paged_attention_mma", "paged_attention_rows"),
+    "feed_forward": ("gemm_glu_fused", "glu_clamped"),
+    "experts": ("moe_grouped", "glu"),
+    "retention_scan": ("retention_scan",),
+    "delta_scan": ("delta_scan",),
+    "sum_and_norm": ("stream_step",),
+}
+SUM_AND_NORM = ("add_rmsnorm",)
+
+
 def design_point(which, z, steps, warmup, clocks, pk):
     """Prefill of 2,048 tokens and decode at batch 8 for one design at one size: tokens a second through
     the engine (recorded passes), and the device time of each kernel entry point in one eager pass."""
@@ -610,7 +667,7 @@ def design_point(which, z, steps, warmup, clocks, pk):
     from kapel_b200.engine import Engine, StepEntry
 
     cfg = {"fusitar": fusitar_config, "kofutar": kofutar_config, "gemma2": gemma_config, "teluzen": teluzen_config, "lokedra": lokedra_config,
-           "mukunex": mukunex_config}[which](z)
+           "mukunex": mukunex_config, "sopalorn": sopalorn_config}[which](z)
     room = (DESIGN_BATCH + 1) * (DESIGN_HISTORY + 4 * (steps + warmup) + 128) + PREFILL_TOKENS
     engine = Engine.random(cfg, seed=0, dtype="bfloat16", max_tokens=room, max_sequences=DESIGN_BATCH + 2)
     rng = np.random.default_rng(0)
@@ -654,12 +711,16 @@ def design_point(which, z, steps, warmup, clocks, pk):
         fn()
         rows = K.timing_report()
         must = design_kernel_rooflines(which, z, kind, PREFILL_TOKENS, DESIGN_HISTORY, DESIGN_BATCH, pk)
+        if which in ("kofutar", "mukunex"):    # a sum in 32-bit in and out, a branch in and the next input out, twice a layer
+            must["sum_and_norm"] = ("bytes", 2 * z["layers"] * (PREFILL_TOKENS if kind == "prefill" else DESIGN_BATCH) * z["width"] * (8 + 2 + 2.0))
         classes = {}
         for name, shape, calls, ms in rows:
             for cls, members in {"kofutar": KOFUTAR_KERNEL_CLASSES, "teluzen": TELUZEN_KERNEL_CLASSES, "lokedra": LOKEDRA_KERNEL_CLASSES,
-                                 "mukunex": MUKUNEX_KERNEL_CLASSES}.get(which, KERNEL_CLASSES).items():
+                                 "mukunex": MUKUNEX_KERNEL_CLASSES, "sopalorn": SOPALORN_KERNEL_CLASSES}.get(which, KERNEL_CLASSES).items():
                 if name in members:
                     classes[cls] = classes.get(cls, 0.0) + ms
+            if which in ("kofutar", "mukunex") and name in SUM_AND_NORM:
+                classes["sum_and_norm"] = classes.get("sum_and_norm", 0.0) + ms
         if which in ("gemma2", "kofutar", "mukunex"):   # the dense way down is a plain product: count the products whose inner width is the intermediate size
             # (Kofutar's input mix has the same shape where the intermediate size is twice the width: one call more than the layers', taken off by its share)
             classes["feed_forward"] = classes.get("feed_forward", 0.0) + sum(
@@ -668,6 +729,9 @@ def design_point(which, z, steps, warmup, clocks, pk):
         if which == "mukunex":             # a parallel layer's output product, over both sides' results, may have the way down's shape: off by its share
             classes["feed_forward"] -= sum(ms * (1.0 - z["layers"] / calls) for name, shape, calls, ms in rows
                                            if name == "gemm" and len(shape) == 2 and shape[0] == z["width"] and shape[1] == z["top"] * z["ff"] and calls > z["layers"])
+        if which == "sopalorn":            # the dense ways down; an output product of as many inner values would be among them
+            classes["feed_forward"] = classes.get("feed_forward", 0.0) + sum(
+                ms for name, shape, calls, ms in rows if name == "gemm" and len(shape) == 2 and shape[0] == z["width"] and shape[1] == z["top"] * z["ff"])
         if which == "teluzen":             # the ways down of the plain layer and of the shared expert
             classes["feed_forward"] = classes.get("feed_forward", 0.0) + sum(
                 ms for name, shape, calls, ms in rows if name == "gemm" and len(shape) == 2 and shape[0] == z["width"] and shape[1] in (z["ff"], z["top"] * z["ff"]))
@@ -698,7 +762,7 @@ def design_line(args) -> int:
     sizes = {}
     for name in args.design_sizes.split(","):
         z = DESIGN_SIZES[name]
-        beside = {"fusitar": ("gemma2",), "lokedra": ("kofutar", "fusitar"), "mukunex": ("kofutar", "lokedra")}.get(args.design, ("fusitar", "gemma2"))
+        beside = {"fusitar": ("gemma2",), "lokedra": ("kofutar", "fusitar"), "mukunex": ("kofutar", "lokedra"), "sopalorn": ("mukunex", "kofutar", "lokedra")}.get(args.design, ("fusitar", "gemma2"))
         if args.design_beside is not None:
             beside = tuple(b for b in args.design_beside.split(",") if b)
         sizes[name] = {"shape": z}
@@ -730,8 +794,8 @@ def main() -> int:
     ap.add_argument("--skip-check", action="store_true", help="leave out the check of the timed logits against the 32-bit path")
     ap.add_argument("--breakdown", action="store_true",
                     help="instead of the JSON line: device time by kernel for one prefill step and one eager decode step")
-    ap.add_argument("--design", default=None, choices=["fusitar", "kofutar", "teluzen", "lokedra", "mukunex"],
-                    help="instead of the default line: this design beside Gemma 2 (kofutar and teluzen: beside Fusitar and Gemma 2; lokedra: beside Kofutar and Fusitar; mukunex: beside Kofutar and Lokedra) at equal sizes, prefill and decode, with each like kernel's roofline fraction")
+    ap.add_argument("--design", default=None, choices=["fusitar", "kofutar", "teluzen", "lokedra", "mukunex", "sopalorn"],
+                    help="instead of the default line: this design beside Gemma 2 (kofutar and teluzen: beside Fusitar and Gemma 2; lokedra: beside Kofutar and Fusitar; mukunex: beside Kofutar and Lokedra; sopalorn: beside Mukunex, Kofutar and Lokedra) at equal sizes, prefill and decode, with each like kernel's roofline fraction")
     ap.add_argument("--design-beside", default=None, help="which other designs run beside it (comma separated; empty: none); default: the closest ones")
     ap.add_argument("--design-sizes", default="s,m", help="which of the design sizes (s, m), comma separated")
     args = ap.parse_args()

@@ -524,7 +524,7 @@ extern "C" int kb_proj_rope_append(const void* src, int src_dt, int splits, long
     const size_t smem = (size_t)(hq + hkv) * d * sizeof(float);
     KB_REQUIRE(smem <= 200 * 1024, "proj_rope_append: rows of %d query and key components do not fit shared memory", (hq + hkv) * d);
     cudaStream_t s = (cudaStream_t)stream;
-    const int threads = (hq + hkv) * d >= 2048 ? 512 : 256;
+    const int threads = (hq + hkv) * d >= 2048 ? (rows <= DEPENDENT_ROWS ? 1024 : 512) : 256;
 #define KB_PRA(TS, TW, TO)                                                                                                      \
     do {                                                                                                                        \
         if (smem > 48 * 1024) cudaFuncSetAttribute(proj_rope_append_kernel<TS, TW, TO>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \

@@ -21,10 +21,60 @@ namespace kb {
 typedef __nv_bfloat16 bf16;
 
 // ------------------------------------------------------------------------------------------ route
-constexpr int ROUTE_THREADS = 256;
+constexpr int ROUTE_THREADS = 256;            // many rows; few rows (a decoding step) take a block of ROUTE_THREADS_FEW: latency counts there
+constexpr int ROUTE_THREADS_FEW = 1024;
+
+// The scores and the choice without groups, by one warp: what thread 0 does below, side by side.
+__device__ __forceinline__ void route_by_warp(float* score, float* choice, const float* __restrict__ correction, int* __restrict__ experts,
+                                              float* __restrict__ weights, int n_experts, int top, int softmax, int renormalize, float scale) {
+    const int lane = threadIdx.x & 31;
+    if (softmax == 1) {
+        float mx = -INFINITY, total = 0.f;
+        for (int x = lane; x < n_experts; x += 32) mx = fmaxf(mx, score[x]);
+        mx = warp_max(mx);
+        for (int x = lane; x < n_experts; x += 32) {
+            score[x] = expf(score[x] - mx);
+            total += score[x];
+        }
+        total = warp_sum(total);
+        for (int x = lane; x < n_experts; x += 32) score[x] /= total;
+    } else if (softmax == 0) {
+        for (int x = lane; x < n_experts; x += 32) score[x] = 1.f / (1.f + expf(-score[x]));
+    }
+    for (int x = lane; x < n_experts; x += 32) choice[x] = score[x] + (correction ? correction[x] : 0.f);
+    __syncwarp();
+    float total = 0.f, first = 0.f;
+    for (int t = 0; t < top; ++t) {
+        int best = 0x7fffffff;
+        float bv = -INFINITY;
+        for (int x = lane; x < n_experts; x += 32)
+            if (choice[x] > bv) { bv = choice[x]; best = x; }
+#pragma unroll
+        for (int o = 16; o > 0; o >>= 1) {                       // the largest; among equals the lowest number
+            const float v = __shfl_xor_sync(0xffffffffu, bv, o);
+            const int b = __shfl_xor_sync(0xffffffffu, best, o);
+            if (v > bv || (v == bv && b < best)) { bv = v; best = b; }
+        }
+        if (best >= n_experts) best = 0;                         // scores that are no numbers: stay in range all the same
+        const float s = score[best];
+        if (t == 0) first = s;
+        total += softmax == 2 ? expf(s - first) : s;
+        if (lane == 0) {
+            experts[t] = best;
+            weights[t] = softmax == 2 ? expf(s - first) : s;
+            choice[best] = -INFINITY;
+        }
+        __syncwarp();
+    }
+    if (softmax == 2 || renormalize || scale != 1.f)
+        for (int t = lane; t < top; t += 32) {
+            const float w = weights[t];
+            weights[t] = (softmax == 2 ? w / total : (renormalize ? w / (total + 1e-20f) : w)) * scale;
+        }
+}
 
 template <typename TH>
-__global__ void __launch_bounds__(ROUTE_THREADS)
+__global__ void __launch_bounds__(ROUTE_THREADS_FEW)
 moe_route_kernel(const TH* __restrict__ h, const float* __restrict__ router, const float* __restrict__ correction,
                  int* __restrict__ experts_out, float* __restrict__ weights_out, int width, int n_experts, int top, int groups,
                  int keep_groups, int group_top, int softmax, int renormalize, float scale) {
@@ -36,7 +86,7 @@ moe_route_kernel(const TH* __restrict__ h, const float* __restrict__ router, con
     const int r = blockIdx.x;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const TH* hr = h + (size_t)r * width;
-    for (int x = warp; x < n_experts; x += ROUTE_THREADS / 32) {
+    for (int x = warp; x < n_experts; x += blockDim.x / 32) {
         const float* w = router + (size_t)x * width;
         // eight loads of each operand ahead of their eight additions, which keep the order of i
         float acc = 0.f;
@@ -55,6 +105,11 @@ moe_route_kernel(const TH* __restrict__ h, const float* __restrict__ router, con
         if (lane == 0) score[x] = acc;
     }
     __syncthreads();
+    if (groups == 1 || keep_groups == groups) {
+        if (warp == 0)
+            route_by_warp(score, choice, correction, experts_out + (size_t)r * top, weights_out + (size_t)r * top, n_experts, top, softmax, renormalize, scale);
+        return;
+    }
     if (threadIdx.x != 0) return;
     if (softmax == 2) {
         // the logits themselves choose; the chosen ones are weighted below
@@ -431,11 +486,12 @@ extern "C" int kb_moe_route(int* experts, float* weights, const void* h, int h_d
     KB_REQUIRE(smem <= 48 * 1024, "moe_route: %d experts are too many for the router's shared memory", n_experts);
     if (rows == 0) return 0;
     cudaStream_t s = (cudaStream_t)stream;
+    const int threads = rows <= DEPENDENT_ROWS ? ROUTE_THREADS_FEW : ROUTE_THREADS;
     if (h_dt == KB_DT_F32)
-        moe_route_kernel<float><<<rows, ROUTE_THREADS, smem, s>>>((const float*)h, router, correction, experts, weights, width, n_experts, top,
+        moe_route_kernel<float><<<rows, threads, smem, s>>>((const float*)h, router, correction, experts, weights, width, n_experts, top,
                                                                   groups, keep_groups, group_top, softmax, renormalize, scale);
     else if (h_dt == KB_DT_BF16)
-        moe_route_kernel<bf16><<<rows, ROUTE_THREADS, smem, s>>>((const bf16*)h, router, correction, experts, weights, width, n_experts, top,
+        moe_route_kernel<bf16><<<rows, threads, smem, s>>>((const bf16*)h, router, correction, experts, weights, width, n_experts, top,
                                                                  groups, keep_groups, group_top, softmax, renormalize, scale);
     else return fail("moe_route: dtype code %d is not known", h_dt);
     return check_launch("moe_route");

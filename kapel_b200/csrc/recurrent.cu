@@ -425,7 +425,7 @@ struct RetentionParams {
 // One block a row, a warp a head: queries, keys and values through the activation, queries and keys turned (component i with
 // i + rotary / 2), keys scaled; the scan's inputs are decay q and k.
 template <typename TS>
-__global__ void __launch_bounds__(256)
+__global__ void __launch_bounds__(1024)
 retention_prep_kernel(const Src<TS> src, const RetentionParams p, const ScanInputs s) {
     const int r = blockIdx.x;
     const size_t base = (size_t)r * p.row_width;
@@ -985,8 +985,9 @@ extern "C" int kb_retention_scan(float* out, float* scratch, const void* src, in
     in.scal = in.val + (size_t)rows * nv;
     in.nv = 2;
     cudaStream_t s = (cudaStream_t)stream;
-    if (in_dt == KB_DT_F32) retention_prep_kernel<float><<<rows, 256, 0, s>>>(Src<float>{(const float*)src, splits, (size_t)split_stride}, g, in);
-    else if (in_dt == KB_DT_BF16) retention_prep_kernel<bf16><<<rows, 256, 0, s>>>(Src<bf16>{(const bf16*)src, splits, (size_t)split_stride}, g, in);
+    const int threads = rows <= DEPENDENT_ROWS ? 1024 : 256;      // few rows: latency counts
+    if (in_dt == KB_DT_F32) retention_prep_kernel<float><<<rows, threads, 0, s>>>(Src<float>{(const float*)src, splits, (size_t)split_stride}, g, in);
+    else if (in_dt == KB_DT_BF16) retention_prep_kernel<bf16><<<rows, threads, 0, s>>>(Src<bf16>{(const bf16*)src, splits, (size_t)split_stride}, g, in);
     else return fail("retention: dtype code %d is not known", in_dt);
     if (int err = check_launch("retention prep")) return err;
     if (by_chunks(longest))

@@ -248,7 +248,7 @@ template <typename TB, typename TH, int V, int SM>
 static int launch_stream_step(const StreamParams& p, const Src<TB>& a, const Src<TB>& b, void* h, int rows, cudaStream_t s) {
     const size_t smem = (size_t)p.width * sizeof(float) * (p.norm_a != nullptr && p.mix != nullptr ? 3 : 1);
     KB_REQUIRE(smem <= 200 * 1024, "stream_step: rows of %d values do not fit the shared memory of a block", p.width);
-    if (smem > 48 * 1024) cudaFuncSetAttribute(stream_step_kernel<TB, TH, V, SM>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    if (smem > 40 * 1024) cudaFuncSetAttribute(stream_step_kernel<TB, TH, V, SM>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     const int chunks = p.width / V;
     const int threads = std::min(STREAM_THREADS, std::max(64, (chunks + 31) / 32 * 32));
     launch_dependent_if(rows <= DEPENDENT_ROWS, stream_step_kernel<TB, TH, V, SM>, dim3(rows), dim3(threads), smem, s, p, a, b, (TH*)h);

@@ -184,7 +184,7 @@ def batch_of(step):
 
 # -------------------------------------------------------------------------------------- streams
 @pytest.mark.parametrize("rows", [3, 70])
-@pytest.mark.parametrize("S,width", [(1, 48), (2, 50), (3, 64), (4, 2052), (5, 33), (8, 320), (11, 76), (16, 20)])
+@pytest.mark.parametrize("S,width", [(1, 48), (2, 50), (3, 64), (4, 2052), (3, 4096), (2, 6001), (5, 33), (8, 320), (11, 76), (16, 20)])
 def test_streams_written_and_read_in_one_kernel(S, width, rows):
     """A branch as a tensor, as partial sums and as two normed branches; with and without a weight a channel; with a layer norm with
     a bias, without one, and an RMS norm; write alone and read alone."""
