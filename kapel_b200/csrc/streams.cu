@@ -45,9 +45,10 @@ template <typename T> struct Pack<1, T> {
     static __device__ __forceinline__ void store(T* p, const float (&v)[1]) { Elem<T>::store(p, v[0]); }
 };
 
-template <int V, typename T>
+template <int V, typename T, bool MANY>
 __device__ __forceinline__ void branch_at(const Src<T>& src, size_t i, float (&v)[V]) {
     Pack<V, T>::load(src.p + i, v);
+    if constexpr (!MANY) return;
     for (int s = 1; s < src.splits; s += 8) {
         float t[8][V];
 #pragma unroll
@@ -96,10 +97,10 @@ __device__ __forceinline__ float2 block_sum2(float a, float b, float* scratch) {
     return make_float2(warp_sum(lane < n ? scratch[lane] : 0.f), warp_sum(lane < n ? scratch[32 + lane] : 0.f));
 }
 
-// SM: room for streams; a thread owns V neighbouring channels of every stream at a time. Shared memory: u [width], and with two
+// SM: room for streams; MANY: branches of more than one slice (a decoding step, as a rule); a thread owns V neighbouring channels of every stream at a time. Shared memory: u [width], and with two
 // normed branches their rows [2 width].
-template <typename TB, typename TH, int V, int SM>
-__global__ void __launch_bounds__(STREAM_THREADS)
+template <typename TB, typename TH, int V, int SM, bool MANY>
+__global__ void __launch_bounds__(STREAM_THREADS, SM <= 4 && !MANY ? 2 : 1)
 stream_step_kernel(const StreamParams p, const Src<TB> a, const Src<TB> b, TH* __restrict__ h) {
     extern __shared__ __align__(16) float row[];
     __shared__ float scratch[64];
@@ -107,44 +108,44 @@ stream_step_kernel(const StreamParams p, const Src<TB> a, const Src<TB> b, TH* _
     const size_t base = (size_t)blockIdx.x * width;
     float* x = p.x + base * S;
     const bool write = p.mix != nullptr, read = p.in != nullptr;
-    // A handful of numbers that every thread needs, constants of the layer: in registers, or in shared memory where there are many.
-    constexpr bool KEEP = SM <= 4;
-    float kept[KEEP ? SM : 1][KEEP ? SM : 1];
-    __shared__ float held[KEEP ? 1 : SM * SM];
-    if constexpr (KEEP) {
-#pragma unroll
-        for (int s = 0; s < SM; ++s)
-#pragma unroll
-            for (int t = 0; t < SM; ++t) kept[s][t] = write && s < S && t < S ? p.mix[s * S + t] : 0.f;
-    } else {
-        for (int i = threadIdx.x; i < SM * SM; i += blockDim.x) held[i] = write && i / SM < S && i % SM < S ? p.mix[i / SM * S + i % SM] : 0.f;
-        __syncthreads();
+    // A handful of numbers that every thread needs, constants of the layer: what goes to stream t lies together.
+    __shared__ __align__(16) float held[SM * SM];
+    __shared__ float out[SM], in[SM];
+    for (int i = threadIdx.x; i < SM * SM; i += blockDim.x) {
+        const int t = i / SM, f = i % SM;
+        held[i] = write && f < S && t < S ? p.mix[f * S + t] : 0.f;
+        if (f == 0) {
+            out[t] = write && t < S ? p.out[t] : 0.f;
+            in[t] = read && t < S ? p.in[t] : 0.f;
+        }
     }
-    auto mix = [&](int s, int t) { if constexpr (KEEP) return kept[s][t]; else return held[s * SM + t]; };
-    float out[SM], in[SM];
-#pragma unroll
-    for (int s = 0; s < SM; ++s) {
-        out[s] = write && s < S ? p.out[s] : 0.f;
-        in[s] = read && s < S ? p.in[s] : 0.f;
-    }
+    __syncthreads();
     dependent_wait();
     dependent_trigger();
-    float inv_a = 0.f, inv_b = 0.f;
     const bool dual = write && p.norm_a != nullptr;
     if (dual) {
         float ssa = 0.f, ssb = 0.f;
         for (int c = threadIdx.x; c < chunks; c += blockDim.x) {
             float va[V], vb[V];
-            branch_at<V, TB>(a, base + (size_t)c * V, va);
-            branch_at<V, TB>(b, base + (size_t)c * V, vb);
+            branch_at<V, TB, MANY>(a, base + (size_t)c * V, va);
+            branch_at<V, TB, MANY>(b, base + (size_t)c * V, vb);
 #pragma unroll
             for (int e = 0; e < V; ++e) { ssa = fmaf(va[e], va[e], ssa); ssb = fmaf(vb[e], vb[e], ssb); }
             Pack<V, float>::store(row + width + c * V, va);
             Pack<V, float>::store(row + 2 * width + c * V, vb);
         }
         const float2 ss = block_sum2(ssa, ssb, scratch);
-        inv_a = 1.f / sqrtf(ss.x / (float)width + p.eps_ab);
-        inv_b = 1.f / sqrtf(ss.y / (float)width + p.eps_ab);
+        const float inv_a = 1.f / sqrtf(ss.x / (float)width + p.eps_ab), inv_b = 1.f / sqrtf(ss.y / (float)width + p.eps_ab);
+        for (int c = threadIdx.x; c < chunks; c += blockDim.x) {        // their sum in the first one's place (this thread's own values)
+            float va[V], vb[V], wa[V], wb[V];
+            Pack<V, float>::load(row + width + c * V, va);
+            Pack<V, float>::load(row + 2 * width + c * V, vb);
+            Pack<V, float>::load(p.norm_a + c * V, wa);
+            Pack<V, float>::load(p.norm_b + c * V, wb);
+#pragma unroll
+            for (int e = 0; e < V; ++e) va[e] = va[e] * inv_a * wa[e] + vb[e] * inv_b * wb[e];
+            Pack<V, float>::store(row + width + c * V, va);
+        }
     }
     float sum = 0.f;
     for (int c = threadIdx.x; c < chunks; c += blockDim.x) {
@@ -158,15 +159,9 @@ stream_step_kernel(const StreamParams p, const Src<TB> a, const Src<TB> b, TH* _
         if (write) {
             float y[V];
             if (dual) {
-                float va[V], vb[V], wa[V], wb[V];
-                Pack<V, float>::load(row + width + c * V, va);
-                Pack<V, float>::load(row + 2 * width + c * V, vb);
-                Pack<V, float>::load(p.norm_a + c * V, wa);
-                Pack<V, float>::load(p.norm_b + c * V, wb);
-#pragma unroll
-                for (int e = 0; e < V; ++e) y[e] = va[e] * inv_a * wa[e] + vb[e] * inv_b * wb[e];
+                Pack<V, float>::load(row + width + c * V, y);
             } else {
-                branch_at<V, TB>(a, base + (size_t)c * V, y);
+                branch_at<V, TB, MANY>(a, base + (size_t)c * V, y);
             }
             if (p.scale != nullptr) {
                 float w[V];
@@ -184,7 +179,7 @@ stream_step_kernel(const StreamParams p, const Src<TB> a, const Src<TB> b, TH* _
                     for (int s = 0; s < SM; ++s)
                         if (s < S) {
 #pragma unroll
-                            for (int e = 0; e < V; ++e) n[e] = fmaf(mix(s, t), v[s][e], n[e]);
+                            for (int e = 0; e < V; ++e) n[e] = fmaf(held[t * SM + s], v[s][e], n[e]);
                         }
                     Pack<V, float>::store(x + (size_t)t * width + c * V, n);
 #pragma unroll
@@ -244,25 +239,28 @@ __global__ void stream_sum_kernel(float* __restrict__ out, const float* __restri
     out[(size_t)i * width + c] = v;
 }
 
-template <typename TB, typename TH, int V, int SM>
+template <typename TB, typename TH, int V, int SM, bool MANY>
 static int launch_stream_step(const StreamParams& p, const Src<TB>& a, const Src<TB>& b, void* h, int rows, cudaStream_t s) {
     const size_t smem = (size_t)p.width * sizeof(float) * (p.norm_a != nullptr && p.mix != nullptr ? 3 : 1);
     KB_REQUIRE(smem <= 200 * 1024, "stream_step: rows of %d values do not fit the shared memory of a block", p.width);
-    if (smem > 40 * 1024) cudaFuncSetAttribute(stream_step_kernel<TB, TH, V, SM>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    if (smem > 40 * 1024) cudaFuncSetAttribute(stream_step_kernel<TB, TH, V, SM, MANY>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     const int chunks = p.width / V;
     const int threads = std::min(STREAM_THREADS, std::max(64, (chunks + 31) / 32 * 32));
-    launch_dependent_if(rows <= DEPENDENT_ROWS, stream_step_kernel<TB, TH, V, SM>, dim3(rows), dim3(threads), smem, s, p, a, b, (TH*)h);
+    launch_dependent_if(rows <= DEPENDENT_ROWS, stream_step_kernel<TB, TH, V, SM, MANY>, dim3(rows), dim3(threads), smem, s, p, a, b, (TH*)h);
     return check_launch("stream_step");
 }
 
 template <typename TB, typename TH>
 static int run_stream_step(const StreamParams& p, const Src<TB>& a, const Src<TB>& b, void* h, int rows, bool wide, cudaStream_t s) {
-#define KB_SS(SM) (wide ? launch_stream_step<TB, TH, 4, SM>(p, a, b, h, rows, s) : launch_stream_step<TB, TH, 1, SM>(p, a, b, h, rows, s))
+    const bool many = a.splits > 1 || b.splits > 1;
+#define KB_SS2(V, SM) (many ? launch_stream_step<TB, TH, V, SM, true>(p, a, b, h, rows, s) : launch_stream_step<TB, TH, V, SM, false>(p, a, b, h, rows, s))
+#define KB_SS(SM) (wide ? KB_SS2(4, SM) : KB_SS2(1, SM))
     if (p.streams <= 2) return KB_SS(2);
     if (p.streams <= 4) return KB_SS(4);
     if (p.streams <= 8) return KB_SS(8);
-    return launch_stream_step<TB, TH, 1, STREAMS_MAX>(p, a, b, h, rows, s);
+    return launch_stream_step<TB, TH, 1, STREAMS_MAX, true>(p, a, b, h, rows, s);
 #undef KB_SS
+#undef KB_SS2
 }
 
 }  // namespace kb
