@@ -355,28 +355,30 @@ def test_attention_with_a_sink_within_a_window_on_every_kernel(way, H, G, d, win
         assert rel_err(attend(way, cache, q, rows, 0.2, np.full(H, 0.5), window), plain_heads(q, k, v, 0.2, np.full(H, 0.5), rows, window)) < 2e-2
 
 
+@pytest.mark.parametrize("window", [77, None])
 @pytest.mark.parametrize("way", WAYS)
-def test_a_windows_edge_and_a_sink_that_show(way):
-    """One key stands out by 20 against a query. Rows that have it just inside their window see it alone (a sink as high halves it), rows
-    that have it just outside do not see it at all, wherever it lies: at the start, at page and tile borders."""
+def test_a_windows_edge_a_far_key_and_a_sink_that_show(way, window):
+    """One key stands out by 20 against a query. Rows that have it just inside their window (without a window: rows hundreds of keys
+    later) see it alone (a sink as high halves it), rows that have it just outside do not see it at all, wherever it lies: at the start,
+    at page and tile borders."""
     rng = np.random.default_rng(3)
     dtype, tol = (torch.float32, 1e-4) if way == "rows f32" else (torch.bfloat16, 3e-2)
-    H, d, T, window = 2, 64, 420, 77
+    H, d, T = 2, 64, 420
     for target in (0, 1, 15, 16, 63, 64, 127, 128, 200, 255, 256, 300):
         k, v = bf16_round(rng.standard_normal((T, 1, d)) * 0.2), bf16_round(rng.standard_normal((T, 1, d)))
         k[:, 0, 0] = 0.0
         k[target, 0] = 0.0
         k[target, 0, 0] = 1.0
-        last = target + window - 1                           # the last row that sees it
+        last = target + window - 1 if window else T - 11     # the last row that sees it, with a window
         rows = list(range(last - 9, last + 11)) if way.startswith("prompt") else [target, last - 1, last, last + 1, last + 2]
         q = bf16_round(rng.standard_normal((len(rows), H, d)) * 0.1)
         q[..., 0] = 20.0
         cache = Paged(rng, k, v, dtype)
         y = attend(way, cache, q, rows, 1.0, np.array([-30.0, 20.0]), window)
-        inside = np.array([r <= last for r in rows])
+        inside = np.array([r <= last or window is None for r in rows])
         assert np.abs(y[inside, 0] - v[target, 0]).max() < tol * 3, target
         assert np.abs(y[inside, 1] - 0.5 * v[target, 0]).max() < tol * 3, target
-        assert np.abs(y[~inside, 1]).max() < 1e-5, target    # without the key the sink takes everything
+        assert window is None or np.abs(y[~inside, 1]).max() < 1e-5, target      # without the key the sink takes everything
         want = plain_heads(q, k, v, 1.0, np.array([-30.0, 20.0]), rows, window)
         assert rel_err(y, want) < tol, target
 
