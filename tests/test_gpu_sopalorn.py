@@ -184,7 +184,7 @@ def batch_of(step):
 
 # -------------------------------------------------------------------------------------- streams
 @pytest.mark.parametrize("rows", [3, 70])
-@pytest.mark.parametrize("S,width", [(1, 48), (2, 50), (3, 64), (4, 2052), (3, 4096), (2, 6001), (5, 33), (8, 320), (11, 76), (16, 20)])
+@pytest.mark.parametrize("S,width", [(1, 48), (2, 50), (3, 64), (4, 2052), (3, 4096), (2, 6001), (5, 33), (8, 264), (11, 76), (16, 20)])
 def test_streams_written_and_read_in_one_kernel(S, width, rows):
     """A branch as a tensor, as partial sums and as two normed branches; with and without a weight a channel; with a layer norm with
     a bias, without one, and an RMS norm; write alone and read alone."""
@@ -335,7 +335,7 @@ def attend(way, cache, q, rows, scale, sinks, window):
 
 
 @pytest.mark.parametrize("way", WAYS)
-@pytest.mark.parametrize("H,G,d,window", [(9, 3, 80, 70), (10, 2, 64, 1), (4, 4, 128, 300), (16, 1, 32, 64), (6, 2, 96, 17), (3, 1, 48, 2000), (6, 3, 96, None)])
+@pytest.mark.parametrize("H,G,d,window", [(9, 3, 80, 70), (10, 2, 64, 1), (4, 4, 128, 300), (16, 1, 32, 64), (8, 2, 112, 19), (3, 1, 48, 2000), (6, 3, 112, None)])
 def test_attention_with_a_sink_within_a_window_on_every_kernel(way, H, G, d, window):
     rng = np.random.default_rng(H * d)
     dtype = torch.float32 if way == "rows f32" else torch.bfloat16
@@ -384,7 +384,7 @@ def test_a_windows_edge_a_far_key_and_a_sink_that_show(way, window):
 
 
 @pytest.mark.parametrize("dtype,tol", [(torch.float32, 1e-5), (torch.bfloat16, 1e-2)])
-@pytest.mark.parametrize("H,d,rotary", [(6, 16, 12), (1, 40, 40), (5, 96, 24), (3, 10, 2)])
+@pytest.mark.parametrize("H,d,rotary", [(6, 16, 12), (1, 40, 40), (5, 72, 20), (3, 10, 2)])
 def test_queries_alone_normed_and_turned(H, d, rotary, dtype, tol):
     """What a layer does that reads another layer's keys: nothing of the cache is touched."""
     from kapel_b200 import kernels as K
@@ -540,7 +540,7 @@ def test_router_with_identity_experts_and_a_scale(experts, identity, top, scale)
 
 
 @pytest.mark.parametrize("rows", [1, 5, 17, 40, 64, 65, 200, 300])
-@pytest.mark.parametrize("n,k", [(40, 64), (384, 320), (1000, 128)])
+@pytest.mark.parametrize("n,k", [(40, 64), (392, 264), (1000, 128)])
 def test_bounded_unit_in_the_products_epilogue(rows, n, k):
     from kapel_b200 import kernels as K
 
